@@ -6,12 +6,14 @@ architecture is added the same way from anywhere: a typed config reader, a build
 crates/hi-mlx/src/config.rs:620-637, crates/hi-mlx/src/models.rs:373-375)."""
 from .config import bezasun as _bezasun
 from .config import fidatar as _fidatar
+from .config import fofisun as _fofisun
 from .config import surinex as _surinex
 from .config import vinurax as _vinurax
 from .config.llama4 import Llama4TextConfig
 from .config.registry import Architecture, register_architecture
 from .parts.bezasun import build_bezasun_spec, normalize_bezasun_tensor_name
 from .parts.fidatar import build_fidatar_spec, normalize_fidatar_tensor_name
+from .parts.fofisun import build_fofisun_spec, normalize_fofisun_tensor_name
 from .parts.llama4 import build_llama4_spec, derive_llama4_tensors, normalize_llama4_tensor_name
 from .parts.surinex import build_surinex_spec, normalize_surinex_tensor_name
 from .parts.vinurax import build_vinurax_spec, normalize_vinurax_tensor_name
@@ -40,3 +42,8 @@ register_architecture(
     ["Bezasun", "bezasun"],
     Architecture(name="bezasun", parse_config=_bezasun.BezasunConfig.from_json, build_spec=build_bezasun_spec,
                  normalize_tensor_name=normalize_bezasun_tensor_name))
+
+register_architecture(
+    ["Fofisun", "fofisun"],
+    Architecture(name="fofisun", parse_config=_fofisun.FofisunConfig.from_json, build_spec=build_fofisun_spec,
+                 normalize_tensor_name=normalize_fofisun_tensor_name))

@@ -46,8 +46,8 @@ def pool_tokens_for_budget(cache_specs: Dict[int, Optional[CacheSpec]], element_
                            portion_tokens: int = 8192) -> List[int]:
     """Pool sizes (tokens per group) from a byte budget (the reference sizes its one pool from the
     token budget of a step, crates/hi-cuda/src/lib.rs:794-797; here the memory that is free decides).
-    A windowed group never holds more than its window, the page being written and the portion in
-    flight for every request, so it gets that (or less, if the budget is smaller); what is left
+    A windowed group never holds more than its window (and the first tokens it keeps), the page being written and the
+    portion in flight for every request, so it gets that (or less, if the budget is smaller); what is left
     goes to the groups that keep every key, in proportion to what a token costs them. ``most_tokens``
     caps the result (``max_requests`` requests at the model's longest context need no more)."""
     groups, _ = plan_groups(cache_specs)
@@ -61,6 +61,8 @@ def pool_tokens_for_budget(cache_specs: Dict[int, Optional[CacheSpec]], element_
     keep_all = [g for g, spec in enumerate(groups) if spec.window is None]
     for g in windowed:
         want = max_requests * (groups[g].window[1] + 2 * page_size) + portion_tokens
+        if groups[g].keep_first:
+            want += max_requests * -(-groups[g].keep_first // page_size) * page_size
         if most_tokens is not None:
             want = min(want, most_tokens)
         share = left // max(1, len(windowed) + len(keep_all)) if keep_all else left // len(windowed)

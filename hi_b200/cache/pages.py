@@ -205,20 +205,21 @@ class CacheManager:
         self.groups = list(groups)
         self.page_size = int(page_size)
         self.max_requests = int(max_requests)
-        kinds, sizes = [], []
+        kinds, sizes, keeps = [], [], []
         for spec in self.groups:
             if spec.window is None:
-                kinds.append(0); sizes.append(0)
+                kinds.append(0); sizes.append(0); keeps.append(0)
             else:
-                kind, size = spec.window
-                if kind not in _WINDOW_KINDS or int(size) <= 0:
+                kind, size = spec.window[:2]
+                if kind not in _WINDOW_KINDS or int(size) <= 0 or spec.keep_first < 0 or \
+                        (spec.keep_first and kind != "sliding"):
                     raise ValueError(f"unknown cache window {spec.window!r}")
-                kinds.append(_WINDOW_KINDS[kind]); sizes.append(int(size))
+                kinds.append(_WINDOW_KINDS[kind]); sizes.append(int(size)); keeps.append(spec.keep_first)
         n = len(self.groups)
         self._lib = host.library()
         self._ptr = self._lib.hbh_cache_create(
             n, (ctypes.c_int * max(n, 1))(*kinds), (ctypes.c_int64 * max(n, 1))(*sizes),
-            (ctypes.c_int * max(n, 1))(*[int(p) for p in pages_per_group]), self.page_size, self.max_requests)
+            (ctypes.c_int64 * max(n, 1))(*keeps), (ctypes.c_int * max(n, 1))(*[int(p) for p in pages_per_group]), self.page_size, self.max_requests)
         if not self._ptr:
             raise ValueError("the native cache manager refused these sizes")
         self._handles = _Handles()

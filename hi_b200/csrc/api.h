@@ -11,6 +11,9 @@ extern "C" {
 int hb_feed_tokens(int* tokens, const int* dst, const int* src, const int* sampled, int n, cudaStream_t stream);
 int hb_embed_gather(const void* table, int table_dtype, const int* tokens, float* out, int n, int hidden,
                     int vocab, float scale, cudaStream_t stream);
+// plus a sinusoidal vector of the position: turns [ceil(hidden / 2)] = frequencies / (2 pi)
+int hb_embed_position(const void* table, int table_dtype, const int* tokens, const int* positions, const double* turns,
+                      float* out, int n, int hidden, int vocab, float scale, cudaStream_t stream);
 // routed_weight (or null): [n * top_k] factors of the routed rows in the sum (a score that scales the
 // experts' outputs). The sum takes x_scale * x; post != 0: the stream takes the normalised row, not the sum.
 int hb_add_rmsnorm(float* x, const void* delta, int delta_dtype, const void* delta2, int delta2_dtype,
@@ -20,6 +23,11 @@ int hb_add_rmsnorm(float* x, const void* delta, int delta_dtype, const void* del
 int hb_swiglu(const void* in, void* out, int dtype, int rows, int inter, cudaStream_t stream);
 int hb_relu2(const void* in, int dtype, void* out, int out_dtype, long long n, cudaStream_t stream);   // max(x, 0)^2
 int hb_convert(const void* in, int dtype, void* out, int out_dtype, long long n, cudaStream_t stream);  // a copy in another dtype
+int hb_gelu(const void* in, void* out, int dtype, long long n, cudaStream_t stream);        // z Phi(z), exact (erf)
+// min(gate, limit) sigmoid(1.702 .) (clamp(up, +-limit) + 1) of rows [gate | up | ...]; scale_col >= 0: times the sigmoid
+// of that column of the row
+int hb_glu_limit(const void* in, long long ld, void* out, int dtype, int rows, int inter, float limit, int scale_col,
+                 cudaStream_t stream);
 int hb_softcap(float* x, float cap, long long n, cudaStream_t stream);                     // cap tanh(x / cap), in place
 int hb_moe_combine(const float* y, const int* slot_of_entry, const float* routed_weight, const void* shared,
                    int shared_dtype, float* out,
@@ -40,10 +48,13 @@ int hb_qkv_post(const void* qkv, int dtype, const float* inv_freq, int rot_pairs
 // p_j = e^{s_j} / (1 + sum e^{s_j}); the term has no value. The general kernel and the merge also take
 // sink_values (float32 [nh] or null): the term's score is the head's own number instead of 0. The general
 // kernel takes softcap (> 0: s <- softcap tanh(s / softcap) after the scale) and slopes (float32 [nh] or null:
-// slopes[h] * (query position - key position) is taken off the score after the cap).
+// slopes[h] * (query position - key position) is taken off the score after the cap). keep (with a window): the first
+// `keep` positions stay visible although the window has passed them. part_acc given and `out` null: the splits'
+// unnormalised rows with their (max, sum) are left in part_acc / part_ml (here, in the decode kernel and in the
+// mma.sync prefill kernel) for a kernel that merges them together with its own work.
 int hb_paged_attention(const void* q, int dtype, const void* k_pages, const void* v_pages,
                        const int* block_table, int table_stride, const int* seq_of_token, const int* positions,
-                       void* out, int n_tokens, int nh, int nkv, int hd, int page_size, int chunk, int window,
+                       void* out, int n_tokens, int nh, int nkv, int hd, int page_size, int chunk, int window, int keep,
                        float scale, int sink, float softcap, const float* slopes, const float* sink_values,
                        int split_size, int max_splits, float* part_acc, float* part_ml, cudaStream_t stream);
 
@@ -51,7 +62,7 @@ int hb_attention_merge(const float* part_acc, const float* part_ml, void* out, i
                        int max_splits, int sink, int nh, const float* sink_values, cudaStream_t stream);
 int hb_attention_decode(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
                         int table_stride, const int* seq_of_token, const int* positions, void* out, int n_tokens,
-                        int nh, int nkv, int hd, int page_size, int chunk, int window, float scale, int sink,
+                        int nh, int nkv, int hd, int page_size, int chunk, int window, int keep, float scale, int sink,
                         const float* head_bias, float softcap, const float* slopes, const float* sink_values,
                         int split_size, int max_splits, float* part_acc, float* part_ml,
                         cudaStream_t stream);   // sink == 2: sigmoid weights with head_bias; plain sums go to part_acc
@@ -76,9 +87,9 @@ int hb_attention_decode_fused(const void* qkv, const float* inv_freq, int rot_pa
 // hb_attention_prefill with reshaped scores: softcap, slopes, sink_values as hb_paged_attention
 int hb_attention_prefill_reshaped(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
                                   int table_stride, const int* cu_seqlens, const int* positions, void* out, int n_seqs,
-                                  int max_new, int nh, int nkv, int hd, int page_size, int chunk, int window, float scale,
-                                  int skip_single, int sink, float softcap, const float* slopes, const float* sink_values,
-                                  cudaStream_t stream);
+                                  int max_new, int nh, int nkv, int hd, int page_size, int chunk, int window, int keep,
+                                  float scale, int skip_single, int sink, float softcap, const float* slopes,
+                                  const float* sink_values, float* part_acc, float* part_ml, cudaStream_t stream);
 int hb_attention_prefill(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
                          int table_stride, const int* cu_seqlens, const int* positions, void* out, int n_seqs,
                          int max_new, int nh, int nkv, int hd, int page_size, int chunk, int window, float scale,
@@ -88,7 +99,7 @@ int hb_attention_prefill(const void* q, const void* k_pages, const void* v_pages
 int hb_attention_prefill_tc_reshaped(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
                                      int table_stride, const int* cu_seqlens, const int* positions, void* out,
                                      int n_tokens, int n_pages, int n_seqs, int max_new, int nh, int nkv, int hd,
-                                     int page_size, int chunk, int window, float scale, int skip_single, int sink,
+                                     int page_size, int chunk, int window, int keep, float scale, int skip_single, int sink,
                                      float softcap, const float* slopes, const float* sink_values, int key_splits,
                                      float* part_acc, float* part_ml, int* status, cudaStream_t stream);
 int hb_attention_prefill_tc(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
@@ -96,6 +107,31 @@ int hb_attention_prefill_tc(const void* q, const void* k_pages, const void* v_pa
                             int n_pages, int n_seqs, int max_new, int nh, int nkv, int hd, int page_size, int chunk,
                             int window, float scale, int skip_single, int sink, const float* head_bias, int key_splits,
                             float* part_acc, float* part_ml, int* status, cudaStream_t stream);   // sink == 2 as above
+// differential attention: both maps of a head in one block, their difference normed and gated in the epilogue
+int hb_diff_prefill_tc(const void* q, const void* k_pages, const void* v_pages, const int* block_table, int table_stride,
+                       const int* cu_seqlens, const int* positions, void* out, int n_tokens, int n_pages, int n_seqs,
+                       int max_new, int nh, int nkv, int hd, int page_size, int chunk, int window, int keep, float scale,
+                       int skip_single, float lambda, float eps, float mul, int vdim, const void* gate,
+                       long long gate_stride, int* status, cudaStream_t stream);
+// differential.cu: the same from split partials [n_rows][2 * heads][splits][hd]; a sigmoid gate alone
+int hb_diff_merge(const float* part_acc, const float* part_ml, const long long* rows, const void* gate,
+                  long long gate_stride, void* out, int dtype, int n_rows, int heads, int hd, int vdim, int splits,
+                  float lambda, float eps, float mul, cudaStream_t stream);
+int hb_gate_rows(const void* o, long long o_stride, const void* gate, long long gate_stride, void* out, int dtype,
+                 long long rows, int heads, int hd, int vdim, cudaStream_t stream);
+// conv_qkv.cu: short causal convolution of the projected q, k, v, norm, rotation, append (one or two maps a head)
+int hb_conv_qkv(const void* proj, int dtype, long long ld, const float* taps, int taps_n, float* state,
+                long long state_stride, long long conv_off, int norm, float eps, const float* q_w, const float* k_w,
+                const float* inv_freq, int rot_pairs, int interleaved, float rot_mul, const int* positions,
+                const int* seq_of_token, const int* cu_seqlens, const int* slots, const int* block_table, int table_stride,
+                void* q_out, void* k_pages, void* v_pages, int page_size, int write_kv, int single_tokens, int n_tokens,
+                int heads, int kv_heads, int maps, int dim, int vdim, int hd, int* moved, cudaStream_t stream);
+// sandwich.cu: stream += norm(sub-layer result), then the norm of the stream
+int hb_sandwich_step(float* x, const void* delta, int delta_dtype, const void* delta2, int delta2_dtype,
+                     const float* routed, const int* slot_of_entry, const float* routed_weight, int top_k,
+                     const float* w_y, float eps_y, const float* w, float eps, void* y, int y_dtype, float* y_f32,
+                     const int* row_map, int rows, int hidden, cudaStream_t stream);
+
 // sigmoid weights, one block per (query tile, head) over all its keys: the block turns its rows back by their
 // positions (values cached rotated: v_inv_freq [v_pairs] or null) and writes `out` (bfloat16) itself
 int hb_sigmoid_prefill_tc(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
@@ -107,17 +143,19 @@ int hb_sigmoid_prefill_tc(const void* q, const void* k_pages, const void* v_page
 // mode: bit 0 = scores are the softmax over all experts (clear: the sigmoid of the chosen logit),
 // bit 1 = the chosen scores are divided by their sum; bits 8-15 = G, 16-23 = KEEP: only experts of the KEEP best
 // of G equal groups of neighbours can be chosen (a group counts as the sum of its two largest sigmoid scores)
-int hb_router_topk(const void* x, int x_dtype, const void* w, int w_dtype, int n, int hidden, int experts,
+// bias (float32 [experts] or null) is added to the logits
+int hb_router_topk(const void* x, int x_dtype, const void* w, int w_dtype, const float* bias, int n, int hidden, int experts,
                    int top_k, int mode, float score_scale, float* logits_out, int* ids, float* scores,
                    cudaStream_t stream);    // score_scale: a constant factor on every chosen score
 int hb_moe_plan(const int* ids, int n_entries, int experts, int* offsets, int* sorted_entry,
                 int* slot_of_entry, int* active, cudaStream_t stream);
-int hb_router_plan(const void* x, int x_dtype, const void* w, int w_dtype, int n, int hidden, int experts, int top_k,
+int hb_router_plan(const void* x, int x_dtype, const void* w, int w_dtype, const float* bias, int n, int hidden, int experts, int top_k,
                    int mode, float score_scale, float* logits_out, int* ids, float* scores, int* offsets,
                    int* sorted_entry, int* slot_of_entry, int* active, int* counter, cudaStream_t stream);
 int hb_moe_gate_up(const void* x, int dtype, const int* sorted_entry, int top_k, const void* w_gate,
                    const void* w_up, const int* offsets, const int* active, int experts, const float* scores,
-                   void* act, int n_entries, int inter, int hidden, int few_rows, int activation, cudaStream_t stream);
+                   void* act, int n_entries, int inter, int hidden, int few_rows, int activation, float limit,
+                   cudaStream_t stream);
 int hb_moe_down(const void* act, int dtype, const void* w_down, const int* offsets, const int* active, int experts,
                 float* y, int n_entries, int hidden, int inter, int few_rows, cudaStream_t stream);
 
@@ -125,7 +163,7 @@ int hb_gather_rows(const void* x, const int* sorted_entry, int top_k, void* xs, 
                    cudaStream_t stream);
 int hb_moe_gate_up_tc(const void* xs, const int* sorted_entry, const void* w_gate, const void* w_up,
                       const int* offsets, int experts, const float* scores, void* act, int rows, int inter,
-                      int hidden, int* status, cudaStream_t stream);
+                      int hidden, float limit, int* status, cudaStream_t stream);
 int hb_moe_down_tc(const void* act, const void* w_down, const int* offsets, int experts, float* y, int rows,
                    int hidden, int inter, float* scratch, long long scratch_floats, int* counters, int n_counters,
                    int* status, cudaStream_t stream);

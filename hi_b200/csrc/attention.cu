@@ -7,6 +7,8 @@
 // result depends only on its own query and the keys it reads: not on how the tokens were
 // cut into steps, on what else is in the batch, or on which pages hold the keys.
 // Scores, max, sum and the weighted sum of values are float32 (models.rs:5963, 6024-6050).
+// With `keep` the first `keep` tokens stay readable although the window has passed them: the keys are then
+// [0, min(keep, lo)) and [lo, p], walked as one run.
 // Query head h reads kv head h / (nh / nkv) (crates/hi-cuda/src/kernels.cu:12413-12414).
 #include "api.h"
 #include "common.cuh"
@@ -19,7 +21,7 @@ __global__ void paged_attention_kernel(const T* __restrict__ q, const T* __restr
                                        const T* __restrict__ v_pages, const int* __restrict__ block_table,
                                        int table_stride, const int* __restrict__ seq_of_token,
                                        const int* __restrict__ positions, T* __restrict__ out, int n_tokens,
-                                       int nh, int nkv, int hd, int page_size, int chunk, int window,
+                                       int nh, int nkv, int hd, int page_size, int chunk, int window, int keep,
                                        float scale, int sink, float softcap, const float* __restrict__ slopes,
                                        const float* __restrict__ sink_values, int split_size, int max_splits,
                                        float* __restrict__ part_acc, float* __restrict__ part_ml) {
@@ -37,18 +39,20 @@ __global__ void paged_attention_kernel(const T* __restrict__ q, const T* __restr
   int lo = 0;
   if (chunk > 0) lo = (pos / chunk) * chunk;
   if (window > 0 && pos - window + 1 > lo) lo = pos - window + 1;
-  // split s of a token covers keys [lo + s*split_size, lo + (s+1)*split_size): a function of the
+  // split s of a token covers its visible keys s*split_size .. (s+1)*split_size - 1: a function of the
   // token's own visible range only, never of the batch
-  int hi = pos;
+  // (visible keys are counted from the first one: number v is key v while v < kept, then key v + skip)
+  const int kept = min(keep, lo), skip = lo - kept;
+  int first = 0, last = pos - skip;
+  const bool parts = part_acc != nullptr;
   if (max_splits > 1) {
     float* ml = part_ml + ((size_t)th * max_splits + split) * 2;
-    const int first = lo + split * split_size;
-    if (first > pos) {
+    first = split * split_size;
+    if (first > last) {
       if (lane == 0) { ml[0] = -INFINITY; ml[1] = 0.f; }
       return;
     }
-    lo = first;
-    hi = min(pos, first + split_size - 1);
+    last = min(last, first + split_size - 1);
   }
 
   float* qs = q_smem + warp * hd;
@@ -63,9 +67,9 @@ __global__ void paged_attention_kernel(const T* __restrict__ q, const T* __restr
   const float slope = slopes ? slopes[h] : 0.f;          // a bias of -slope * (distance to the key)
   const float inv_cap = softcap > 0.f ? 1.f / softcap : 0.f;
 
-  for (int base = lo; base <= hi; base += 32) {
-    const int key = base + lane;
-    const bool valid = key <= hi;
+  for (int base = first; base <= last; base += 32) {
+    const int key = base + lane < kept ? base + lane : base + lane + skip;
+    const bool valid = base + lane <= last;
     float s = -INFINITY;
     int page = -1;
     if (valid) {
@@ -91,12 +95,12 @@ __global__ void paged_attention_kernel(const T* __restrict__ q, const T* __restr
     l = l * corr + hb::warp_sum(p);
 #pragma unroll
     for (int i = 0; i < kMaxDimsPerLane; ++i) acc[i] *= corr;
-    const int count = min(32, hi - base + 1);
+    const int count = min(32, last - base + 1);
     for (int j = 0; j < count; ++j) {
       const float pj = __shfl_sync(0xffffffffu, p, j);
       const int pg = __shfl_sync(0xffffffffu, page, j);
-      if (pg < 0) continue;
-      const T* vrow = v_pages + (((size_t)pg * nkv + kvh) * page_size + ((base + j) % page_size)) * hd;
+      if (pg < 0) continue;            // the same for every lane
+      const T* vrow = v_pages + (((size_t)pg * nkv + kvh) * page_size + (__shfl_sync(0xffffffffu, key, j) % page_size)) * hd;
 #pragma unroll
       for (int i = 0; i < kMaxDimsPerLane; ++i) {
         const int d = lane + 32 * i;
@@ -105,7 +109,7 @@ __global__ void paged_attention_kernel(const T* __restrict__ q, const T* __restr
     }
     m = m_new;
   }
-  if (max_splits > 1) {
+  if (parts) {
     float* pa = part_acc + ((size_t)th * max_splits + split) * hd;
 #pragma unroll
     for (int i = 0; i < kMaxDimsPerLane; ++i) {
@@ -189,16 +193,18 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_acc, const
 
 }  // namespace
 
+// `part_acc` null: one pass per (token, head) into `out`. Otherwise the splits' partial rows go to part_acc / part_ml
+// and are merged into `out`, or (`out` null) left there for a kernel that merges them with what it does next.
 extern "C" int hb_paged_attention(const void* q, int dtype, const void* k_pages, const void* v_pages,
                                   const int* block_table, int table_stride, const int* seq_of_token,
                                   const int* positions, void* out, int n_tokens, int nh, int nkv, int hd,
-                                  int page_size, int chunk, int window, float scale, int sink, float softcap,
+                                  int page_size, int chunk, int window, int keep, float scale, int sink, float softcap,
                                   const float* slopes, const float* sink_values, int split_size,
                                   int max_splits, float* part_acc, float* part_ml, cudaStream_t stream) {
-  if (!q || !k_pages || !v_pages || !block_table || !seq_of_token || !positions || !out) return HB_ERR_BAD_ARG;
-  if (max_splits < 1 || (max_splits > 1 && (split_size <= 0 || !part_acc || !part_ml))) return HB_ERR_BAD_ARG;
+  if (!q || !k_pages || !v_pages || !block_table || !seq_of_token || !positions || (!out && !part_acc)) return HB_ERR_BAD_ARG;
+  if (max_splits < 1 || (max_splits > 1 && (split_size <= 0 || !part_acc)) || (part_acc && !part_ml)) return HB_ERR_BAD_ARG;
   if (n_tokens < 0 || nh <= 0 || nkv <= 0 || nh % nkv != 0 || page_size <= 0 || table_stride <= 0 ||
-      chunk < 0 || window < 0)
+      chunk < 0 || window < 0 || keep < 0)
     return HB_ERR_BAD_ARG;
   if (hd <= 0 || hd % 8 != 0 || hd > 1024) return HB_ERR_UNSUPPORTED;
   const bool wide = hd > 256, widest = hd > 512;
@@ -211,7 +217,7 @@ extern "C" int hb_paged_attention(const void* q, int dtype, const void* k_pages,
 #define HB_PAGED_ATTENTION(T, DPL)                                                                              \
   paged_attention_kernel<T, DPL><<<(int)blocks, warps_per_block * 32, smem, stream>>>(                          \
       (const T*)q, (const T*)k_pages, (const T*)v_pages, block_table, table_stride, seq_of_token, positions,    \
-      (T*)out, n_tokens, nh, nkv, hd, page_size, chunk, window, scale, sink, softcap, slopes, sink_values, split_size,   \
+      (T*)out, n_tokens, nh, nkv, hd, page_size, chunk, window, keep, scale, sink, softcap, slopes, sink_values, split_size,   \
       max_splits, part_acc, part_ml)
   if (dtype == HB_DTYPE_F32) {
     if (widest) HB_PAGED_ATTENTION(float, 32); else if (wide) HB_PAGED_ATTENTION(float, 16); else HB_PAGED_ATTENTION(float, 8);
@@ -224,7 +230,7 @@ extern "C" int hb_paged_attention(const void* q, int dtype, const void* k_pages,
   }
 #undef HB_PAGED_ATTENTION
   HB_LAUNCH_CHECK();
-  if (max_splits > 1) {
+  if (part_acc && out) {
     if (dtype == HB_DTYPE_F32)
       attention_merge_kernel<float><<<n_tokens * nh, 128, (max_splits + 33) * sizeof(float), stream>>>(part_acc, part_ml, (float*)out, hd, max_splits, sink, nh, sink_values);
     else

@@ -9,6 +9,9 @@
 // memory with cp.async (double-buffered); each of the 4 warps takes 16 keys of a tile and keeps
 // its own running max / sum / output, merged in warp order at the end. Partials (m, l, acc) go
 // to scratch and are merged across splits by attention_merge (attention.cu).
+// A window that keeps the first tokens of a request (`keep`) is walked in tiles of 64 positions, first the tiles of the
+// kept tokens that lie before the window, then the window's; a split is then a fixed run of tiles of that walk.
+// More than 16 query heads on a kv head are cut into row tiles of 16, one block each (grid y).
 #include <cuda_bf16.h>
 
 #include "api.h"
@@ -54,7 +57,7 @@ __global__ void __launch_bounds__(NWARPS * 32)
 attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pages,
                    const __nv_bfloat16* __restrict__ v_pages, const int* __restrict__ block_table,
                    int table_stride, const int* __restrict__ seq_of_token, const int* __restrict__ positions,
-                   __nv_bfloat16* __restrict__ out, int nh, int nkv, int page_size, int chunk, int window,
+                   __nv_bfloat16* __restrict__ out, int nh, int nkv, int page_size, int chunk, int window, int keep,
                    float scale, int sink, const float* __restrict__ head_bias, float softcap,
                    const float* __restrict__ slopes, const float* __restrict__ sink_values, int split_size,
                    int max_splits, float* __restrict__ part_acc, float* __restrict__ part_ml) {
@@ -72,28 +75,42 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
   float* ml_s = reinterpret_cast<float*>(v_s + 2 * TILE * STRIDE);              // [NWARPS][ROWS][2]
   float* o_s = reinterpret_cast<float*>(k_s);   // [ROWS][HD], reuses the K tiles once the key loop is over
 
-  const int split = blockIdx.x, kvh = blockIdx.y, t = blockIdx.z;
+  const int row_tiles = (nh / nkv + ROWS - 1) / ROWS;
+  const int split = blockIdx.x, kvh = blockIdx.y / row_tiles, t = blockIdx.z;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int G = nh / nkv;
+  const int row0 = (blockIdx.y % row_tiles) * ROWS;           // first head of the group in this block's row tile
+  const int G = min(ROWS, nh / nkv - row0);                   // heads of the row tile
+  const int h0 = kvh * (nh / nkv) + row0;
+  const bool parts = part_acc != nullptr;
   const int pos = positions[t];
   const int* table = block_table + (size_t)seq_of_token[t] * table_stride;
   int lo = 0;
   if (chunk > 0) lo = (pos / chunk) * chunk;
   if (window > 0 && pos - window + 1 > lo) lo = pos - window + 1;
   const int first = lo + split * split_size;
-  const size_t th0 = (size_t)t * nh + (size_t)kvh * G;      // (token, first head of the group)
-  if (first > pos) {                                          // this token has fewer splits
+  const size_t th0 = (size_t)t * nh + h0;                     // (token, first head of the row tile)
+  // kept tokens: tiles of the walk that lie before the window's first tile, this split's first tile, tiles in all
+  const int kept_tiles = keep > 0 ? min((keep + TILE - 1) / TILE, lo / TILE) : 0;
+  const int walk0 = split * (split_size / TILE);
+  const int walk_tiles = kept_tiles + pos / TILE - lo / TILE + 1;
+  if (keep > 0 ? walk0 >= walk_tiles : first > pos) {         // this token has fewer splits
     if (sigmoid) {
       for (int i = tid; i < G * HD; i += NWARPS * 32)
         part_acc[((th0 + i / HD) * max_splits + split) * HD + i % HD] = 0.f;
-    } else if (max_splits > 1 && tid < G) {
+    } else if (parts && tid < G) {
       float* ml = part_ml + ((th0 + tid) * max_splits + split) * 2;
       ml[0] = -INFINITY; ml[1] = 0.f;
     }
     return;
   }
-  const int last = min(pos, first + split_size - 1);
-  const int n_tiles = (last - first + TILE) / TILE;
+  const int last = keep > 0 ? pos : min(pos, first + split_size - 1);
+  const int n_tiles = keep > 0 ? min(split_size / TILE, walk_tiles - walk0) : (last - first + TILE) / TILE;
+  auto tile_base = [&](int tile) {
+    if (keep <= 0) return first + tile * TILE;
+    const int w = walk0 + tile;
+    return (w < kept_tiles ? w : lo / TILE + w - kept_tiles) * TILE;
+  };
+  auto visible = [&](int key) { return key <= last && (keep <= 0 || key >= lo || key < keep); };
 
   // the query rows of this kv group
   for (int c = tid; c < ROWS * CHUNKS; c += NWARPS * 32) {
@@ -104,9 +121,9 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
   // thread -> every 128th 16-byte chunk of a [TILE][CHUNKS] tile. When a tile never straddles a page (page_size
   // a multiple of TILE and the range starts on a TILE boundary) one table lookup serves the whole tile.
   static_assert((TILE * CHUNKS) % (NWARPS * 32) == 0, "whole passes of the block");
-  const bool tile_in_page = (page_size % TILE == 0) && (first % TILE == 0);
+  const bool tile_in_page = (page_size % TILE == 0) && (keep > 0 || first % TILE == 0);
   auto load_tile = [&](int tile, int buf) {
-    const int base = first + tile * TILE;
+    const int base = tile_base(tile);
     __nv_bfloat16* kd = k_s + buf * TILE * STRIDE;
     __nv_bfloat16* vd = v_s + buf * TILE * STRIDE;
     if (tile_in_page) {
@@ -148,14 +165,14 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
   unsigned q_frag[HD / 16][4];
   float row_bias[2] = {0.f, 0.f}, row_slope[2] = {0.f, 0.f};
   if (slopes) {
-    if (lane / 4 < G) row_slope[0] = slopes[kvh * G + lane / 4];
-    if (lane / 4 + 8 < G) row_slope[1] = slopes[kvh * G + lane / 4 + 8];
+    if (lane / 4 < G) row_slope[0] = slopes[h0 + lane / 4];
+    if (lane / 4 + 8 < G) row_slope[1] = slopes[h0 + lane / 4 + 8];
   }
   const bool reshaped = softcap > 0.f || slopes != nullptr;
   const float inv_cap = softcap > 0.f ? 1.f / softcap : 0.f;
   if (sigmoid && head_bias) {
-    if (lane / 4 < G) row_bias[0] = head_bias[kvh * G + lane / 4];
-    if (lane / 4 + 8 < G) row_bias[1] = head_bias[kvh * G + lane / 4 + 8];
+    if (lane / 4 < G) row_bias[0] = head_bias[h0 + lane / 4];
+    if (lane / 4 + 8 < G) row_bias[1] = head_bias[h0 + lane / 4 + 8];
   }
 
   for (int tile = 0; tile < n_tiles; ++tile) {
@@ -185,7 +202,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
       mma_bf16(s_acc[1], q_frag[ks], b[2], b[3]);
     }
     // scale, mask keys past the split's end, online softmax per row (rows lane/4 and lane/4 + 8)
-    const int key0 = first + tile * TILE + warp * 16 + (lane % 4) * 2;
+    const int key0 = tile_base(tile) + warp * 16 + (lane % 4) * 2;
     unsigned p_frag[4];
     if (sigmoid) {
       float p[2][4];
@@ -194,7 +211,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int key = key0 + nt * 8 + (e & 1);
-          p[nt][e] = key <= last ? 1.f / (1.f + __expf(-(s_acc[nt][e] * scale + row_bias[e >> 1]))) : 0.f;
+          p[nt][e] = visible(key) ? 1.f / (1.f + __expf(-(s_acc[nt][e] * scale + row_bias[e >> 1]))) : 0.f;
         }
       p_frag[0] = pack_bf16(p[0][0], p[0][1]);
       p_frag[1] = pack_bf16(p[0][2], p[0][3]);
@@ -207,8 +224,9 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int key = key0 + nt * 8 + (e & 1);
-          float v = key <= last ? s_acc[nt][e] * scale : -INFINITY;
-          if (reshaped && key <= last) {
+          const bool vis = visible(key);
+          float v = vis ? s_acc[nt][e] * scale : -INFINITY;
+          if (reshaped && vis) {
             if (softcap > 0.f) v = softcap * tanhf(v * inv_cap);
             v -= row_slope[e >> 1] * (float)(pos - key);
           }
@@ -315,7 +333,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
     const float o = o_s[row * HD + d];
     if (sigmoid) {
       part_acc[((th0 + row) * max_splits + split) * HD + d] = o;
-    } else if (max_splits > 1) {
+    } else if (parts) {
       part_acc[((th0 + row) * max_splits + split) * HD + d] = o;
       if (d == 0) {
         float* ml = part_ml + ((th0 + row) * max_splits + split) * 2;
@@ -323,7 +341,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
       }
     } else {
       // a key without a value, of score 0 or of the head's own score
-      if (sink && l > 0.f) l += expf((sink_values ? sink_values[kvh * G + row] : 0.f) - mx);
+      if (sink && l > 0.f) l += expf((sink_values ? sink_values[h0 + row] : 0.f) - mx);
       out[(th0 + row) * HD + d] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
     }
   }
@@ -333,7 +351,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
 template <int HD>
 int launch_decode(const void* q, const void* k_pages, const void* v_pages, const int* block_table, int table_stride,
                   const int* seq_of_token, const int* positions, void* out, int n_tokens, int nh, int nkv,
-                  int page_size, int chunk, int window, float scale, int sink, const float* head_bias, float softcap,
+                  int page_size, int chunk, int window, int keep, float scale, int sink, const float* head_bias, float softcap,
                   const float* slopes, const float* sink_values, int split_size,
                   int max_splits, float* part_acc, float* part_ml, cudaStream_t stream) {
   constexpr int STRIDE = HD + 8;
@@ -342,10 +360,10 @@ int launch_decode(const void* q, const void* k_pages, const void* v_pages, const
   static_assert(2 * TILE * STRIDE * sizeof(__nv_bfloat16) >= ROWS * HD * sizeof(float), "o_s aliases the K tiles");
   cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
-  dim3 grid(max_splits, nkv, n_tokens);
+  dim3 grid(max_splits, nkv * ((nh / nkv + ROWS - 1) / ROWS), n_tokens);
   attn_decode_kernel<HD><<<grid, NWARPS * 32, smem, stream>>>(
       (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, block_table, table_stride,
-      seq_of_token, positions, (__nv_bfloat16*)out, nh, nkv, page_size, chunk, window, scale, sink, head_bias, softcap,
+      seq_of_token, positions, (__nv_bfloat16*)out, nh, nkv, page_size, chunk, window, keep, scale, sink, head_bias, softcap,
       slopes, sink_values, split_size, max_splits, part_acc, part_ml);
   HB_LAUNCH_CHECK();
   return HB_OK;
@@ -353,32 +371,34 @@ int launch_decode(const void* q, const void* k_pages, const void* v_pages, const
 
 }  // namespace
 
-// bfloat16 only; head_dim 64, 128 or 192; at most 16 query heads per kv head; every token is taken
-// as one decode row. Returns HB_ERR_UNSUPPORTED for other shapes (the caller then uses the
+// bfloat16 only; head_dim 64, 128 or 192; every token is taken as one decode row. `part_acc` null (one split): the rows
+// go to `out`; otherwise (max, sum, unnormalised row) of every split go to part_ml / part_acc and `out` is not used.
+// With `keep` > 0 (a sliding window only) `split_size * max_splits` has to cover the walk: at most
+// ceil((window + 63) / 64) + ceil(keep / 64) tiles of 64. Returns HB_ERR_UNSUPPORTED for other shapes (the caller then uses the
 // general kernel). The merge over splits is hb_attention_merge.
 extern "C" int hb_attention_decode(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
                                    int table_stride, const int* seq_of_token, const int* positions, void* out,
-                                   int n_tokens, int nh, int nkv, int hd, int page_size, int chunk, int window,
+                                   int n_tokens, int nh, int nkv, int hd, int page_size, int chunk, int window, int keep,
                                    float scale, int sink, const float* head_bias, float softcap, const float* slopes,
                                    const float* sink_values, int split_size, int max_splits,
                                    float* part_acc, float* part_ml, cudaStream_t stream) {
   if (sink == 2 && (softcap > 0.f || slopes || sink_values)) return HB_ERR_UNSUPPORTED;
-  if (!q || !k_pages || !v_pages || !block_table || !seq_of_token || !positions || !out) return HB_ERR_BAD_ARG;
+  if (!q || !k_pages || !v_pages || !block_table || !seq_of_token || !positions || (!out && !part_acc)) return HB_ERR_BAD_ARG;
   if (n_tokens < 0 || nh <= 0 || nkv <= 0 || nh % nkv != 0 || page_size <= 0 || table_stride <= 0 || chunk < 0 ||
-      window < 0 || max_splits < 1 || split_size <= 0 || split_size % TILE != 0)
+      window < 0 || keep < 0 || (keep > 0 && window <= 0) || max_splits < 1 || split_size <= 0 || split_size % TILE != 0)
     return HB_ERR_BAD_ARG;
-  if (sink == 2 ? !part_acc : (max_splits > 1 && (!part_acc || !part_ml))) return HB_ERR_BAD_ARG;
-  if (nh / nkv > ROWS || n_tokens > 65535 || nkv > 65535) return HB_ERR_UNSUPPORTED;
+  if (sink == 2 ? !part_acc : ((max_splits > 1 && !part_acc) || (part_acc && !part_ml))) return HB_ERR_BAD_ARG;
+  if (n_tokens > 65535 || (long long)nkv * ((nh / nkv + ROWS - 1) / ROWS) > 65535) return HB_ERR_UNSUPPORTED;
   if (n_tokens == 0) return HB_OK;
   if (hd == 192)
     return launch_decode<192>(q, k_pages, v_pages, block_table, table_stride, seq_of_token, positions, out, n_tokens,
-                              nh, nkv, page_size, chunk, window, scale, sink, head_bias, softcap, slopes, sink_values, split_size, max_splits, part_acc, part_ml, stream);
+                              nh, nkv, page_size, chunk, window, keep, scale, sink, head_bias, softcap, slopes, sink_values, split_size, max_splits, part_acc, part_ml, stream);
   if (hd == 128)
     return launch_decode<128>(q, k_pages, v_pages, block_table, table_stride, seq_of_token, positions, out, n_tokens,
-                              nh, nkv, page_size, chunk, window, scale, sink, head_bias, softcap, slopes, sink_values, split_size, max_splits, part_acc, part_ml, stream);
+                              nh, nkv, page_size, chunk, window, keep, scale, sink, head_bias, softcap, slopes, sink_values, split_size, max_splits, part_acc, part_ml, stream);
   if (hd == 64)
     return launch_decode<64>(q, k_pages, v_pages, block_table, table_stride, seq_of_token, positions, out, n_tokens,
-                             nh, nkv, page_size, chunk, window, scale, sink, head_bias, softcap, slopes, sink_values, split_size, max_splits, part_acc, part_ml, stream);
+                             nh, nkv, page_size, chunk, window, keep, scale, sink, head_bias, softcap, slopes, sink_values, split_size, max_splits, part_acc, part_ml, stream);
   return HB_ERR_UNSUPPORTED;
 }
 
@@ -452,7 +472,7 @@ extern "C" int hb_attention_decode_static(const void* q, const void* k_pages, co
     if (rc != HB_OK) return rc;
   }
   int rc = hb_attention_decode(q, k_pages, v_pages, block_table, table_stride, seq_of_token, positions, out, n_tokens,
-                               nh, nkv, hd, page_size, chunk, window, scale, 0, nullptr, 0.f, nullptr, nullptr, split_size, max_splits, acc, ml, stream);
+                               nh, nkv, hd, page_size, chunk, window, 0, scale, 0, nullptr, 0.f, nullptr, nullptr, split_size, max_splits, acc, ml, stream);
   if (rc != HB_OK || max_splits == 1 || n_tokens == 0) return rc;
   return hb_attention_merge(acc, ml, out, HB_DTYPE_BF16, n_tokens * nh, hd, max_splits, 0, nh, nullptr, stream);
 }

@@ -7,6 +7,9 @@
 //   through shared memory with cp.async (double-buffered) from the pages the block table names.
 // Masks are by absolute position: key <= query, key >= the query's chunk start / window start.
 // A token's result depends on its own row and keys only (tiles are walked in position order).
+// keep > 0: the first `keep` positions stay visible although the window has passed them; their tiles come first.
+// part_acc [rows][nh][hd] / part_ml [rows][nh][2] (or null): rows leave unnormalised in float32 with their max and sum
+// instead of going to `out`.
 #include "api.h"
 #include "common.cuh"
 #include "mma.cuh"
@@ -22,9 +25,9 @@ __global__ void __launch_bounds__(NWARPS * 32)
 attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pages,
                     const __nv_bfloat16* __restrict__ v_pages, const int* __restrict__ block_table,
                     int table_stride, const int* __restrict__ cu_seqlens, const int* __restrict__ positions,
-                    __nv_bfloat16* __restrict__ out, int nh, int nkv, int page_size, int chunk, int window,
+                    __nv_bfloat16* __restrict__ out, int nh, int nkv, int page_size, int chunk, int window, int keep,
                     float scale, int skip_single, int sink, float softcap, const float* __restrict__ slopes,
-                    const float* __restrict__ sink_values) {
+                    const float* __restrict__ sink_values, float* __restrict__ part_acc, float* __restrict__ part_ml) {
   // softcap > 0: a scaled score s becomes softcap * tanh(s / softcap); slopes [nh]: slopes[head] * (distance to the
   // key) is taken off after the cap; sink_values [nh]: the sink's score is the head's own number instead of 0.
   constexpr int STRIDE = HD + 8;
@@ -53,6 +56,9 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   };
   const int tile_begin = first_visible(p_first) / TILE;    // lo grows with the position
   const int tile_end = p_last / TILE;                      // inclusive
+  const int kept_tiles = keep > 0 ? min((keep + TILE - 1) / TILE, tile_begin) : 0;
+  const int n_tiles = kept_tiles + tile_end - tile_begin + 1;
+  auto tile_at = [&](int i) { return i < kept_tiles ? i : tile_begin + i - kept_tiles; };
   const bool tile_in_page = (page_size % TILE) == 0;
 
   // the query rows, then tiles of keys and values: thread -> every 128th 16-byte chunk of the [rows][CHUNKS] tile
@@ -94,7 +100,7 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
       }
     }
   };
-  load_tile(tile_begin, 0);
+  load_tile(tile_at(0), 0);
   hb::cp_async_commit();
 
   // this thread's two rows of the warp's 16 (mma C layout): g and g + 8
@@ -115,17 +121,18 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     for (int e = 0; e < 4; ++e) o_acc[j][e] = 0.f;
   unsigned q_frag[HD / 16][4];
 
-  for (int kt = tile_begin; kt <= tile_end; ++kt) {
-    const int buf = (kt - tile_begin) & 1;
-    if (kt < tile_end) {
-      load_tile(kt + 1, buf ^ 1);
+  for (int it = 0; it < n_tiles; ++it) {
+    const int kt = tile_at(it);
+    const int buf = it & 1;
+    if (it + 1 < n_tiles) {
+      load_tile(tile_at(it + 1), buf ^ 1);
       hb::cp_async_commit();
       hb::cp_async_wait<1>();
     } else {
       hb::cp_async_wait<0>();
     }
     __syncthreads();
-    if (kt == tile_begin) {
+    if (it == 0) {
 #pragma unroll
       for (int ks = 0; ks < HD / 16; ++ks)
         hb::ldmatrix_x4(q_frag[ks], q_s + (warp * 16 + (lane % 16)) * STRIDE + ks * 16 + (lane / 16) * 8);
@@ -158,7 +165,8 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
         for (int e = 0; e < 4; ++e) {
           const int key = key0 + nt * 8 + (e & 1);
           const bool second = e >> 1;
-          const bool vis = second ? (ok_b && key <= pos_b && key >= lo_b) : (ok_a && key <= pos_a && key >= lo_a);
+          const bool vis = second ? (ok_b && key <= pos_b && (key >= lo_b || key < keep))
+                                  : (ok_a && key <= pos_a && (key >= lo_a || key < keep));
           float v = vis ? s_acc[nt][e] * scale : -INFINITY;
           if (reshaped && vis) {
             if (softcap > 0.f) v = softcap * tanhf(v * inv_cap);
@@ -219,6 +227,21 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     }
     __syncthreads();
   }
+  if (part_acc) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      if (!(r ? ok_b : ok_a)) continue;
+      const size_t at = (size_t)(tok0 + (r ? rb : ra)) * nh + h;
+      if (lane % 4 == 0) {
+        part_ml[at * 2] = m_run[r];
+        part_ml[at * 2 + 1] = l_run[r];
+      }
+#pragma unroll
+      for (int j = 0; j < HD / 8; ++j)
+        *reinterpret_cast<float2*>(part_acc + at * HD + j * 8 + (lane % 4) * 2) = make_float2(o_acc[j][2 * r], o_acc[j][2 * r + 1]);
+    }
+    return;
+  }
   if (sink) {      // one more term in the denominator, of score 0 or of the head's own score; it has no value
     const float sv = sink_values ? sink_values[h] : 0.f;
     if (l_run[0] > 0.f) l_run[0] += expf(sv - m_run[0]);
@@ -241,8 +264,8 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
 template <int HD>
 int launch_prefill(const void* q, const void* k_pages, const void* v_pages, const int* block_table, int table_stride,
                    const int* cu_seqlens, const int* positions, void* out, int n_seqs, int max_new, int nh, int nkv,
-                   int page_size, int chunk, int window, float scale, int skip_single, int sink, float softcap,
-                   const float* slopes, const float* sink_values, cudaStream_t stream) {
+                   int page_size, int chunk, int window, int keep, float scale, int skip_single, int sink, float softcap,
+                   const float* slopes, const float* sink_values, float* part_acc, float* part_ml, cudaStream_t stream) {
   constexpr int STRIDE = HD + 8;
   const size_t smem = (size_t)(BQ * STRIDE + 4 * TILE * STRIDE) * sizeof(__nv_bfloat16);
   cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -250,8 +273,8 @@ int launch_prefill(const void* q, const void* k_pages, const void* v_pages, cons
   dim3 grid((max_new + BQ - 1) / BQ, nh, n_seqs);
   attn_prefill_kernel<HD><<<grid, NWARPS * 32, smem, stream>>>(
       (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, block_table, table_stride,
-      cu_seqlens, positions, (__nv_bfloat16*)out, nh, nkv, page_size, chunk, window, scale, skip_single, sink, softcap,
-      slopes, sink_values);
+      cu_seqlens, positions, (__nv_bfloat16*)out, nh, nkv, page_size, chunk, window, keep, scale, skip_single, sink, softcap,
+      slopes, sink_values, part_acc, part_ml);
   HB_LAUNCH_CHECK();
   return HB_OK;
 }
@@ -264,9 +287,11 @@ int launch_prefill(const void* q, const void* k_pages, const void* v_pages, cons
 extern "C" int hb_attention_prefill_reshaped(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
                                     int table_stride, const int* cu_seqlens, const int* positions, void* out,
                                     int n_seqs, int max_new, int nh, int nkv, int hd, int page_size, int chunk,
-                                    int window, float scale, int skip_single, int sink, float softcap,
-                                             const float* slopes, const float* sink_values, cudaStream_t stream) {
-  if (!q || !k_pages || !v_pages || !block_table || !cu_seqlens || !positions || !out) return HB_ERR_BAD_ARG;
+                                    int window, int keep, float scale, int skip_single, int sink, float softcap,
+                                             const float* slopes, const float* sink_values, float* part_acc, float* part_ml,
+                                             cudaStream_t stream) {
+  if (!q || !k_pages || !v_pages || !block_table || !cu_seqlens || !positions || (!out && !part_acc)) return HB_ERR_BAD_ARG;
+  if (keep < 0 || (keep > 0 && window <= 0) || (part_acc && !part_ml)) return HB_ERR_BAD_ARG;
   if (n_seqs < 0 || max_new < 0 || nh <= 0 || nkv <= 0 || nh % nkv != 0 || page_size <= 0 || table_stride <= 0 ||
       chunk < 0 || window < 0)
     return HB_ERR_BAD_ARG;
@@ -274,13 +299,13 @@ extern "C" int hb_attention_prefill_reshaped(const void* q, const void* k_pages,
   if (n_seqs == 0 || max_new == 0) return HB_OK;
   if (hd == 192)
     return launch_prefill<192>(q, k_pages, v_pages, block_table, table_stride, cu_seqlens, positions, out, n_seqs,
-                               max_new, nh, nkv, page_size, chunk, window, scale, skip_single, sink, softcap, slopes, sink_values, stream);
+                               max_new, nh, nkv, page_size, chunk, window, keep, scale, skip_single, sink, softcap, slopes, sink_values, part_acc, part_ml, stream);
   if (hd == 128)
     return launch_prefill<128>(q, k_pages, v_pages, block_table, table_stride, cu_seqlens, positions, out, n_seqs,
-                               max_new, nh, nkv, page_size, chunk, window, scale, skip_single, sink, softcap, slopes, sink_values, stream);
+                               max_new, nh, nkv, page_size, chunk, window, keep, scale, skip_single, sink, softcap, slopes, sink_values, part_acc, part_ml, stream);
   if (hd == 64)
     return launch_prefill<64>(q, k_pages, v_pages, block_table, table_stride, cu_seqlens, positions, out, n_seqs,
-                              max_new, nh, nkv, page_size, chunk, window, scale, skip_single, sink, softcap, slopes, sink_values, stream);
+                              max_new, nh, nkv, page_size, chunk, window, keep, scale, skip_single, sink, softcap, slopes, sink_values, part_acc, part_ml, stream);
   return HB_ERR_UNSUPPORTED;
 }
 
@@ -289,6 +314,6 @@ extern "C" int hb_attention_prefill(const void* q, const void* k_pages, const vo
                                     int n_seqs, int max_new, int nh, int nkv, int hd, int page_size, int chunk,
                                     int window, float scale, int skip_single, int sink, cudaStream_t stream) {
   return hb_attention_prefill_reshaped(q, k_pages, v_pages, block_table, table_stride, cu_seqlens, positions, out, n_seqs,
-                                       max_new, nh, nkv, hd, page_size, chunk, window, scale, skip_single, sink, 0.f, nullptr,
-                                       nullptr, stream);
+                                       max_new, nh, nkv, hd, page_size, chunk, window, 0, scale, skip_single, sink, 0.f, nullptr,
+                                       nullptr, nullptr, nullptr, stream);
 }

@@ -16,6 +16,10 @@
 //               moved, and writes P as bfloat16 back into tensor memory (tcgen05.st): the products
 //               are bound by what the SM can read from shared memory, and P from there would add a
 //               fifth to it.
+// Differential attention (two maps per head over the same values, maps == 2): one block = 64 new tokens of one request
+// and BOTH maps of a head. Row r of the tile is token r % 64 of map r / 64, so the two maps share every key and value
+// tile, and the epilogue subtracts them, norms the head's row and gates it before it leaves (see Pair).
+// A window that keeps the first tokens of a request (keep > 0) walks the tiles of the kept tokens first.
 // Every mbarrier wait is bounded; on a time-out a code goes to `status` and the block leaves
 // through the common exit, where tensor memory is freed.
 #include <cuda.h>
@@ -38,6 +42,16 @@ __device__ __forceinline__ float fast_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+
+// What the epilogue does with the two maps a1, a2 of a head (float32, normalised by their softmax):
+//   o = a1 - lambda a2;  o <- o rsqrt(mean over vdim of o^2 + eps) mul;  out = o * sigmoid(gate)   (gate null: no gate)
+// `out` is [rows, nh / 2, vdim]; gate row t starts at gate + t * gate_stride and is laid out as a row of `out`.
+struct Pair {
+  float lambda, eps, mul;
+  int vdim, vec;                 // vec: vdim, the rows of `out` and of the gate allow 16-byte accesses
+  const __nv_bfloat16* gate;
+  long long gate_stride;
+};
 
 struct Args {
   const int* block_table;
@@ -72,9 +86,11 @@ struct Args {
   // With a distance bias the newest keys score highest: the key tiles are then taken newest first, so that the running
   // maximum is found in the first tiles and O is seldom rescaled (oldest first it would move with nearly every tile).
   int newest_first;
+  int keep;                  // a sliding window's kept first tokens
+  Pair pair;                 // kPair only
 };
 
-template <int HD>
+template <int HD, bool kPair>
 __global__ void __launch_bounds__(THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, const Args a) {
@@ -109,17 +125,20 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
   uint64_t* s_free = bars + 13;       // 2
   uint64_t* p_ready = bars + 15;      // 1
   uint64_t* pv_done = bars + 16;      // 1
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 17);
+  uint64_t* ex_ready = bars + 17;     // 1   kPair: the maps' halves, then their sums of squares, are in shared memory
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 18);
   constexpr int kst = KST;
+  constexpr int TOKENS = kPair ? BQ / 2 : BQ;   // new tokens of a block
 
   // Blocks start in the order x, y, z: the heads are x and the query tiles y, latest first, so
   // the tiles that read the most keys start first for every head and the short ones fill the end.
-  const int seq = blockIdx.z, h = blockIdx.x % a.nh, piece = blockIdx.x / a.nh;
+  const int heads = kPair ? a.nh / 2 : a.nh;
+  const int seq = blockIdx.z, h = blockIdx.x % heads, piece = blockIdx.x / heads;
   const int qt = gridDim.y - 1 - blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seq_begin = a.cu_seqlens[seq], seq_end = a.cu_seqlens[seq + 1];
-  const int tok0 = seq_begin + qt * BQ;
-  const int n_valid = min(BQ, seq_end - tok0);
+  const int tok0 = seq_begin + qt * TOKENS;
+  const int n_valid = min(TOKENS, seq_end - tok0);
   if (n_valid <= 0) return;
   // a row that this block leaves out weighs nothing in the merge
   const bool sigmoid = a.sink == 2;
@@ -133,7 +152,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     if (a.key_splits > 1 && threadIdx.x == 0) no_part(0);
     return;
   }
-  const int kvh = h / (a.nh / a.nkv);
+  const int kvh = (kPair ? 2 * h : h) / (a.nh / a.nkv);
   const int p_first = a.positions[tok0];
   const int p_last = p_first + n_valid - 1;
   auto first_visible = [&](int pos) {
@@ -143,7 +162,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     return lo;
   };
   int tile_begin = first_visible(p_first) / BKEYS;
-  int nt = p_last / BKEYS - tile_begin + 1;
+  // the walk: tiles of kept tokens before the window's first tile, then the window's
+  const int kept_tiles = a.keep > 0 ? min((a.keep + BKEYS - 1) / BKEYS, tile_begin) : 0;
+  int nt = kept_tiles + p_last / BKEYS - tile_begin + 1;
   if (a.key_splits > 1) {                       // this block's share of the key tiles
     const int share = (nt + a.key_splits - 1) / a.key_splits;
     tile_begin += piece * share;
@@ -153,6 +174,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
       return;
     }
   }
+  auto tile_key0 = [&](int j) {                 // first key position of the j-th tile of this block
+    const int w = a.newest_first ? nt - 1 - j : j;
+    return (w < kept_tiles ? w : tile_begin + w - kept_tiles) * BKEYS;
+  };
 
   if (threadIdx.x == 0) {
     tc::mbar_init(q_full, 1);
@@ -163,6 +188,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     }
     tc::mbar_init(p_ready, 4);
     tc::mbar_init(pv_done, 1);
+    tc::mbar_init(ex_ready, 4);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   if (warp == 1) {
@@ -178,14 +204,20 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     if (lane == 0) {                            // ---- TMA producer
       const int* table = a.block_table + (size_t)seq * a.table_stride;
       tc::mbar_expect_tx(q_full, QBYTES);
-      for (int c = 0; c < DBLK; ++c) tc::tma_load_2d(q_s + c * QBLOCK, &map_q, h * HD + c * 64, tok0, q_full);
+      if (kPair) {                              // the box is 64 rows: map 1 above map 2 in every 64-element block
+        for (int c = 0; c < DBLK; ++c)
+          for (int mp = 0; mp < 2; ++mp)
+            tc::tma_load_2d(q_s + c * QBLOCK + mp * (QBLOCK / 2), &map_q, (2 * h + mp) * HD + c * 64, tok0, q_full);
+      } else {
+        for (int c = 0; c < DBLK; ++c) tc::tma_load_2d(q_s + c * QBLOCK, &map_q, h * HD + c * 64, tok0, q_full);
+      }
       const int boxes = BKEYS / a.box_rows;
       bool ok = true;
       // one tile of K or V: a box per page
       auto load = [&](int j, uint8_t* dst, const CUtensorMap* map, uint64_t* full) {
         tc::mbar_expect_tx(full, KBYTES);
         for (int b = 0; b < boxes; ++b) {
-          const int key0 = (a.newest_first ? tile_begin + nt - 1 - j : tile_begin + j) * BKEYS + b * a.box_rows;
+          const int key0 = tile_key0(j) + b * a.box_rows;
           const int page = key0 <= p_last ? table[key0 / a.page_size] : -1;
           // keys past the portion's last position (or without a page) are masked: any row will do
           const int row = page >= 0 ? (page * a.nkv + kvh) * a.page_size + key0 % a.page_size : 0;
@@ -255,8 +287,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     const int quarter = warp & 3;
     const int r = quarter * 32 + lane;
     const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
-    const bool row_ok = r < n_valid;
-    const int pos = p_first + r;
+    const int row = kPair ? r % TOKENS : r;     // this row's token within the block
+    const int warp_row = kPair ? (quarter & 1) * 32 : quarter * 32;
+    const bool row_ok = row < n_valid;
+    const int pos = p_first + row;
     const int lo = first_visible(pos);
     float m = -INFINITY, l = 0.f;
     const float bias_log2 = (sigmoid && a.head_bias) ? a.head_bias[h] * 1.4426950408889634f : 0.f;
@@ -275,11 +309,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         break;
       }
       tc::fence_after();
-      const int key_base = (a.newest_first ? tile_begin + nt - 1 - j : tile_begin + j) * BKEYS;
+      const int key_base = tile_key0(j);
       // a tile every row of this warp sees whole needs no masks (most tiles of a long prompt)
-      const int warp_first_pos = p_first + quarter * 32;
-      const bool interior = (quarter * 32 + 31 < n_valid) && (key_base + BKEYS - 1 <= warp_first_pos) &&
-                            (key_base >= first_visible(warp_first_pos + 31));
+      const int warp_first_pos = p_first + warp_row;
+      const bool interior = (warp_row + 31 < n_valid) && (key_base + BKEYS - 1 <= warp_first_pos) &&
+                            (key_base >= first_visible(warp_first_pos + 31) || key_base + BKEYS <= a.keep);
       float sv[BKEYS];
       float mx = m;
       {
@@ -323,7 +357,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         for (int i = 0; i < BKEYS; ++i) {
           const int key = key_base + i;
           // masked scores become -inf BEFORE scaling, so the same exponential code serves both paths
-          const float s = (row_ok && key <= pos && key >= lo) ? sv[i] : -INFINITY;
+          const float s = (row_ok && key <= pos && (key >= lo || key < a.keep)) ? sv[i] : -INFINITY;
           sv[i] = s;
           mx = fmaxf(mx, s * scale_l2);
         }
@@ -436,7 +470,86 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         if (lane == 0) atomicExch(a.status, 18);
       } else {
         tc::fence_after();
-        if (sigmoid && a.turn_inside) {
+        if constexpr (kPair) {
+          // The maps trade halves through shared memory (the K tiles are through): row (token, map 1) finishes the
+          // first half of the head's values, row (token, map 2) the second; their sums of squares meet there too.
+          constexpr int HALF = HD / 2, EXS = HALF + 1;
+          float* ex = reinterpret_cast<float*>(k_s);           // [2 maps][64 tokens][EXS]
+          float* ex_ss = ex + 2 * TOKENS * EXS;                // [2][64]
+          static_assert((2 * TOKENS * EXS + 2 * TOKENS) * 4 <= KST * KBYTES, "the exchange fits the K tiles");
+          const int mp = r / TOKENS;
+          const float inv = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll 1
+          for (int c = 0; c < HALF; c += 32) {
+            float o[32];
+            tc::ld32(tmem_o + lane_addr + (1 - mp) * HALF + c, o);
+#pragma unroll
+            for (int i = 0; i < 32; ++i) ex[(mp * TOKENS + row) * EXS + c + i] = o[i] * inv;
+          }
+          __syncwarp();
+          if (lane == 0) tc::mbar_arrive(ex_ready);
+          bool met = __all_sync(0xffffffffu, tc::mbar_wait(ex_ready, 0));
+          float v[HALF];
+          float ss = 0.f;
+          if (met) {
+#pragma unroll
+            for (int c = 0; c < HALF; c += 32) {
+              float o[32];
+              tc::ld32(tmem_o + lane_addr + mp * HALF + c, o);
+#pragma unroll
+              for (int i = 0; i < 32; ++i) {
+                const float mine = o[i] * inv, other = ex[((1 - mp) * TOKENS + row) * EXS + c + i];
+                const float d = mp == 0 ? mine - a.pair.lambda * other : other - a.pair.lambda * mine;
+                v[c + i] = d;
+                ss += d * d;
+              }
+            }
+            ex_ss[mp * TOKENS + row] = ss;
+            __syncwarp();
+            if (lane == 0) tc::mbar_arrive(ex_ready);
+            met = __all_sync(0xffffffffu, tc::mbar_wait(ex_ready, 1));
+          }
+          if (!met) {
+            if (lane == 0) atomicExch(a.status, 23);
+          } else if (row_ok) {
+            const float total = ex_ss[row] + ex_ss[TOKENS + row];
+            const float mul = rsqrtf(total / (float)a.pair.vdim + a.pair.eps) * a.pair.mul;
+            __nv_bfloat16* dst = a.out + ((size_t)(tok0 + row) * heads + h) * a.pair.vdim;
+            const __nv_bfloat16* gate =
+                a.pair.gate ? a.pair.gate + (size_t)(tok0 + row) * a.pair.gate_stride + (size_t)h * a.pair.vdim : nullptr;
+#pragma unroll
+            for (int c = 0; c < HALF; c += 8) {
+              const int d0 = mp * HALF + c;
+              if (d0 >= a.pair.vdim) continue;
+              float g[8];
+              if (a.pair.vec) {                 // vdim is a multiple of 8: the run is whole
+                if (gate) hb::load8(gate + d0, g);
+              } else if (gate) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) g[e] = d0 + e < a.pair.vdim ? __bfloat162float(gate[d0 + e]) : 0.f;
+              }
+#pragma unroll
+              for (int e = 0; e < 8; ++e) {
+                v[c + e] *= mul;
+                if (gate) v[c + e] *= __fdividef(1.f, 1.f + __expf(-g[e]));
+              }
+              if (a.pair.vec) {
+                uint4 pack;
+                uint32_t* w = reinterpret_cast<uint32_t*>(&pack);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                  __nv_bfloat162 hh = __floats2bfloat162_rn(v[c + 2 * e], v[c + 2 * e + 1]);
+                  w[e] = *reinterpret_cast<uint32_t*>(&hh);
+                }
+                *reinterpret_cast<uint4*>(dst + d0) = pack;
+              } else {
+#pragma unroll
+                for (int e = 0; e < 8; ++e)
+                  if (d0 + e < a.pair.vdim) dst[d0 + e] = __float2bfloat16_rn(v[c + e]);
+              }
+            }
+          }
+        } else if (sigmoid && a.turn_inside) {
           // the plain sum is the result: turned back by the row's position in float32, rounded once
           __nv_bfloat16* dst = a.out + ((size_t)(tok0 + r) * a.nh + h) * HD;
           const float fpos = (float)pos;
@@ -544,22 +657,23 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
   }
 }
 
-template <int HD>
+template <int HD, bool kPair = false>
 int launch(const void* q, const void* k_pages, const void* v_pages, const Args& a, int n_tokens, long long pool_rows,
            int n_seqs, int max_new, cudaStream_t stream) {
   CUtensorMap mq, mk, mv;
-  if (!tc::make_map_bf16(&mq, q, (uint64_t)n_tokens, (uint64_t)a.nh * HD, BQ) ||
+  if (!tc::make_map_bf16(&mq, q, (uint64_t)n_tokens, (uint64_t)a.nh * HD, kPair ? BQ / 2 : BQ) ||
       !tc::make_map_bf16(&mk, k_pages, (uint64_t)pool_rows, HD, a.box_rows) ||
       !tc::make_map_bf16(&mv, v_pages, (uint64_t)pool_rows, HD, a.box_rows))
     return HB_ERR_UNSUPPORTED;
   const size_t smem = (size_t)BQ * HD * 2 + (KST + 2) * (size_t)BKEYS * HD * 2 + 256;
-  cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD, kPair>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
-  const int q_tiles = (max_new + BQ - 1) / BQ;
+  const int tokens = kPair ? BQ / 2 : BQ;
+  const int q_tiles = (max_new + tokens - 1) / tokens;
   if (q_tiles > 65535 || n_seqs > 65535) return HB_ERR_UNSUPPORTED;
   if ((long long)a.nh * a.key_splits > 0x7fffffffLL) return HB_ERR_UNSUPPORTED;
-  dim3 grid(a.nh * a.key_splits, q_tiles, n_seqs);
-  attn_prefill_tc_kernel<HD><<<grid, THREADS, smem, stream>>>(mq, mk, mv, a);
+  dim3 grid((kPair ? a.nh / 2 : a.nh) * a.key_splits, q_tiles, n_seqs);
+  attn_prefill_tc_kernel<HD, kPair><<<grid, THREADS, smem, stream>>>(mq, mk, mv, a);
   HB_LAUNCH_CHECK();
   return HB_OK;
 }
@@ -578,7 +692,7 @@ int prefill_tc(const void* q, const void* k_pages, const void* v_pages, const in
                int nh, int nkv, int hd, int page_size, int chunk, int window, float scale, int skip_single, int sink,
                const float* head_bias, int key_splits, float* part_acc, float* part_ml, int* status, int turn_inside,
                const float* v_inv_freq, int v_pairs, int v_interleaved, float softcap, const float* slopes,
-               const float* sink_values, cudaStream_t stream);
+               const float* sink_values, int keep, const Pair* pair, cudaStream_t stream);
 }  // namespace
 
 extern "C" int hb_attention_prefill_tc(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
@@ -589,7 +703,7 @@ extern "C" int hb_attention_prefill_tc(const void* q, const void* k_pages, const
                                        float* part_ml, int* status, cudaStream_t stream) {
   return prefill_tc(q, k_pages, v_pages, block_table, table_stride, cu_seqlens, positions, out, n_tokens, n_pages, n_seqs,
                     max_new, nh, nkv, hd, page_size, chunk, window, scale, skip_single, sink, head_bias, key_splits,
-                    part_acc, part_ml, status, 0, nullptr, 0, 0, 0.f, nullptr, nullptr, stream);
+                    part_acc, part_ml, status, 0, nullptr, 0, 0, 0.f, nullptr, nullptr, 0, nullptr, stream);
 }
 
 // The same with reshaped scores (see Args): a cap, a distance bias per head, a sink with a score per head.
@@ -597,12 +711,12 @@ extern "C" int hb_attention_prefill_tc_reshaped(const void* q, const void* k_pag
                                                 const int* block_table, int table_stride, const int* cu_seqlens,
                                                 const int* positions, void* out, int n_tokens, int n_pages, int n_seqs,
                                                 int max_new, int nh, int nkv, int hd, int page_size, int chunk,
-                                                int window, float scale, int skip_single, int sink, float softcap,
+                                                int window, int keep, float scale, int skip_single, int sink, float softcap,
                                                 const float* slopes, const float* sink_values, int key_splits,
                                                 float* part_acc, float* part_ml, int* status, cudaStream_t stream) {
   return prefill_tc(q, k_pages, v_pages, block_table, table_stride, cu_seqlens, positions, out, n_tokens, n_pages, n_seqs,
                     max_new, nh, nkv, hd, page_size, chunk, window, scale, skip_single, sink, nullptr, key_splits,
-                    part_acc, part_ml, status, 0, nullptr, 0, 0, softcap, slopes, sink_values, stream);
+                    part_acc, part_ml, status, 0, nullptr, 0, 0, softcap, slopes, sink_values, keep, nullptr, stream);
 }
 
 // Sigmoid weights with the result written by the kernel itself: `out` [n_tokens, nh, hd] bfloat16 takes every
@@ -619,7 +733,26 @@ extern "C" int hb_sigmoid_prefill_tc(const void* q, const void* k_pages, const v
   if (v_pairs > 0 && !v_interleaved && 2 * v_pairs != hd) return HB_ERR_UNSUPPORTED;
   return prefill_tc(q, k_pages, v_pages, block_table, table_stride, cu_seqlens, positions, out, n_tokens, n_pages, n_seqs,
                     max_new, nh, nkv, hd, page_size, chunk, window, scale, skip_single, 2, head_bias, 1, nullptr, nullptr,
-                    status, 1, v_inv_freq, v_pairs, v_interleaved, 0.f, nullptr, nullptr, stream);
+                    status, 1, v_inv_freq, v_pairs, v_interleaved, 0.f, nullptr, nullptr, 0, nullptr, stream);
+}
+
+// Differential attention: q [n_tokens, nh, hd] holds the two maps of head a as heads 2a and 2a + 1, both over the same
+// key and value rows of kv head 2a / (nh / nkv) (a map's query is zero where the row belongs to the other map's key).
+// out [n_tokens, nh / 2, vdim] bfloat16 = (a1 - lambda a2) rsqrt(mean(.^2) + eps) mul, times sigmoid(gate) where
+// `gate` (bfloat16, row t at gate + t * gate_stride, nh / 2 * vdim wide) is given. Rows of requests that `skip_single`
+// leaves out are not written.
+extern "C" int hb_diff_prefill_tc(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
+                                  int table_stride, const int* cu_seqlens, const int* positions, void* out, int n_tokens,
+                                  int n_pages, int n_seqs, int max_new, int nh, int nkv, int hd, int page_size, int chunk,
+                                  int window, int keep, float scale, int skip_single, float lambda, float eps, float mul,
+                                  int vdim, const void* gate, long long gate_stride, int* status, cudaStream_t stream) {
+  if (nh % 2 != 0 || nkv <= 0 || (nh / nkv) % 2 != 0 || vdim <= 0 || vdim > hd || (gate && gate_stride < (long long)(nh / 2) * vdim))
+    return HB_ERR_BAD_ARG;
+  const bool vec = vdim % 8 == 0 && ((uintptr_t)out & 15) == 0 && (!gate || (((uintptr_t)gate & 15) == 0 && gate_stride % 8 == 0));
+  const Pair pair{lambda, eps, mul, vdim, vec ? 1 : 0, (const __nv_bfloat16*)gate, gate_stride};
+  return prefill_tc(q, k_pages, v_pages, block_table, table_stride, cu_seqlens, positions, out, n_tokens, n_pages, n_seqs,
+                    max_new, nh, nkv, hd, page_size, chunk, window, scale, skip_single, 0, nullptr, 1, nullptr, nullptr,
+                    status, 0, nullptr, 0, 0, 0.f, nullptr, nullptr, keep, &pair, stream);
 }
 
 namespace {
@@ -628,21 +761,28 @@ int prefill_tc(const void* q, const void* k_pages, const void* v_pages, const in
                int nh, int nkv, int hd, int page_size, int chunk, int window, float scale, int skip_single, int sink,
                const float* head_bias, int key_splits, float* part_acc, float* part_ml, int* status, int turn_inside,
                const float* v_inv_freq, int v_pairs, int v_interleaved, float softcap, const float* slopes,
-               const float* sink_values, cudaStream_t stream) {
+               const float* sink_values, int keep, const Pair* pair, cudaStream_t stream) {
   if (sink == 2 && (softcap > 0.f || slopes || sink_values)) return HB_ERR_UNSUPPORTED;
   if (!q || !k_pages || !v_pages || !block_table || !cu_seqlens || !positions || !out || !status) return HB_ERR_BAD_ARG;
   if (n_tokens < 0 || n_pages <= 0 || n_seqs < 0 || max_new < 0 || nh <= 0 || nkv <= 0 || nh % nkv != 0 ||
       page_size <= 0 || table_stride <= 0 || chunk < 0 || window < 0 || key_splits < 1 || key_splits > 64 ||
-      (sink == 2 && !turn_inside ? !part_acc : (key_splits > 1 && (!part_acc || !part_ml))))
+      keep < 0 || (keep > 0 && window <= 0) || (sink == 2 && !turn_inside ? !part_acc : (key_splits > 1 && (!part_acc || !part_ml))))
     return HB_ERR_BAD_ARG;
+  if (keep > 0 && key_splits > 1) return HB_ERR_UNSUPPORTED;
   if (page_size % 16 != 0 || !(BKEYS % page_size == 0 || page_size % BKEYS == 0)) return HB_ERR_UNSUPPORTED;
   if (n_seqs > 65535 || nh > 65535) return HB_ERR_UNSUPPORTED;
   if (!(scale > 0.f)) return HB_ERR_UNSUPPORTED;       // the largest raw score is taken for the largest scaled one
   if (n_seqs == 0 || max_new == 0 || n_tokens == 0) return HB_OK;
   Args a{block_table, cu_seqlens, positions, (__nv_bfloat16*)out, status, table_stride, nh, nkv, page_size, chunk,
          window, skip_single, page_size < BKEYS ? page_size : BKEYS, scale * 1.4426950408889634f, key_splits, part_acc, part_ml, sink, head_bias,
-         turn_inside, v_pairs, v_interleaved, v_inv_freq, softcap, slopes, sink_values, slopes ? 1 : 0};
+         turn_inside, v_pairs, v_interleaved, v_inv_freq, softcap, slopes, sink_values, slopes ? 1 : 0, keep, pair ? *pair : Pair{}};
   const long long pool_rows = (long long)n_pages * nkv * page_size;
+  if (pair) {
+    if (hd == 192) return launch<192, true>(q, k_pages, v_pages, a, n_tokens, pool_rows, n_seqs, max_new, stream);
+    if (hd == 128) return launch<128, true>(q, k_pages, v_pages, a, n_tokens, pool_rows, n_seqs, max_new, stream);
+    if (hd == 64) return launch<64, true>(q, k_pages, v_pages, a, n_tokens, pool_rows, n_seqs, max_new, stream);
+    return HB_ERR_UNSUPPORTED;
+  }
   if (hd == 192) return launch<192>(q, k_pages, v_pages, a, n_tokens, pool_rows, n_seqs, max_new, stream);
   if (hd == 128) return launch<128>(q, k_pages, v_pages, a, n_tokens, pool_rows, n_seqs, max_new, stream);
   if (hd == 64) return launch<64>(q, k_pages, v_pages, a, n_tokens, pool_rows, n_seqs, max_new, stream);

@@ -28,6 +28,12 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(flo
   return __float2bfloat16_rn(v);
 }
 
+// a gated unit with limits: g = min(gate, limit), u = clamp(up, +-limit), g sigmoid(1.702 g) (u + 1)
+__device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -178,6 +178,25 @@ __global__ void moe_combine_kernel(const float* y, const int* slot_of_entry, con
   }
 }
 
+// The same with a sinusoidal vector of the token's position added after the scale: entry 2i is sin(p f_i), entry 2i + 1
+// cos(p f_i). turns[i] = f_i / (2 pi) in double: the angle is reduced to a fraction of a turn before it is rounded, so
+// that it is exact to float32 at any position.
+__global__ void embed_position_kernel(const void* table, int table_dtype, const int* tokens, const int* positions,
+                                      const double* turns, float* out, int hidden, int vocab, float scale) {
+  const int t = blockIdx.y;
+  const int id = tokens[t];
+  const bool ok = id >= 0 && id < vocab;
+  const double pos = (double)positions[t];
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; 2 * i < hidden; i += gridDim.x * blockDim.x) {
+    const double turn = pos * turns[i];
+    float sn, cs;
+    sincospif(2.f * (float)(turn - rint(turn)), &sn, &cs);
+    const size_t at = (size_t)id * hidden + 2 * i, to = (size_t)t * hidden + 2 * i;
+    out[to] = (ok ? load_any(table, table_dtype, at) * scale : 0.f) + sn;
+    if (2 * i + 1 < hidden) out[to + 1] = (ok ? load_any(table, table_dtype, at + 1) * scale : 0.f) + cs;
+  }
+}
+
 bool dtype_ok(int d) { return d == HB_DTYPE_F32 || d == HB_DTYPE_BF16; }
 
 }  // namespace
@@ -189,6 +208,22 @@ extern "C" int hb_embed_gather(const void* table, int table_dtype, const int* to
   if (n == 0) return HB_OK;
   embed_gather_kernel<<<n, 256, 0, stream>>>(table, table_dtype, tokens, out, hidden, vocab, scale);
   HB_LAUNCH_CHECK();
+  return HB_OK;
+}
+
+extern "C" int hb_embed_position(const void* table, int table_dtype, const int* tokens, const int* positions,
+                                 const double* turns, float* out, int n, int hidden, int vocab, float scale,
+                                 cudaStream_t stream) {
+  if (!table || !tokens || !positions || !turns || !out || n < 0 || hidden <= 0 || vocab <= 0 || !dtype_ok(table_dtype))
+    return HB_ERR_BAD_ARG;
+  if (n > 65535 * 8) return HB_ERR_UNSUPPORTED;
+  if (n == 0) return HB_OK;
+  for (int first = 0; first < n; first += 65535) {
+    const int here = n - first < 65535 ? n - first : 65535;
+    embed_position_kernel<<<dim3(((hidden + 1) / 2 + 255) / 256, here), 256, 0, stream>>>(
+        table, table_dtype, tokens + first, positions + first, turns, out + (size_t)first * hidden, hidden, vocab, scale);
+    HB_LAUNCH_CHECK();
+  }
   return HB_OK;
 }
 
@@ -343,6 +378,98 @@ extern "C" int hb_relu2(const void* in, int dtype, void* out, int out_dtype, lon
   if (n == 0) return HB_OK;
   const long long want = (n / 4 + 255) / 256 + 1;
   relu2_kernel<<<(int)(want < 148 * 16 ? want : 148 * 16), 256, 0, stream>>>(in, dtype, out, out_dtype, (size_t)n);
+  HB_LAUNCH_CHECK();
+  return HB_OK;
+}
+
+// out = z Phi(z), Phi the normal distribution's cumulative function: 0.5 z (1 + erf(z / sqrt 2)); n % 8 == 0
+template <typename T>
+__global__ void gelu8_kernel(const T* __restrict__ in, T* __restrict__ out, size_t groups) {
+  for (size_t g = (size_t)blockIdx.x * blockDim.x + threadIdx.x; g < groups; g += (size_t)gridDim.x * blockDim.x) {
+    float v[8];
+    hb::load8(in + 8 * g, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = 0.5f * v[e] * (1.f + erff(v[e] * 0.70710678118654752f));
+#pragma unroll
+    for (int e = 0; e < 8; e += 4)
+      store4_any(out, sizeof(T) == 4 ? HB_DTYPE_F32 : HB_DTYPE_BF16, 8 * g + e, make_float4(v[e], v[e + 1], v[e + 2], v[e + 3]));
+  }
+}
+
+__global__ void gelu_kernel(const void* __restrict__ in, void* __restrict__ out, int dtype, size_t n) {
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+    const float v = load_any(in, dtype, i);
+    store_any(out, dtype, i, 0.5f * v * (1.f + erff(v * 0.70710678118654752f)));
+  }
+}
+
+extern "C" int hb_gelu(const void* in, void* out, int dtype, long long n, cudaStream_t stream) {
+  if (!in || !out || n < 0 || !dtype_ok(dtype)) return HB_ERR_BAD_ARG;
+  if (n == 0) return HB_OK;
+  const long long want = ((n % 8 == 0 ? n / 8 : n) + 255) / 256;
+  const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
+  if (n % 8 != 0) gelu_kernel<<<blocks, 256, 0, stream>>>(in, out, dtype, (size_t)n);
+  else if (dtype == HB_DTYPE_F32) gelu8_kernel<float><<<blocks, 256, 0, stream>>>((const float*)in, (float*)out, (size_t)n / 8);
+  else gelu8_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)in, (__nv_bfloat16*)out, (size_t)n / 8);
+  HB_LAUNCH_CHECK();
+  return HB_OK;
+}
+
+// Clamped gate: g = min(in[t, j], limit), u = clamp(in[t, inter + j], +-limit), out[t, j] = g sigmoid(1.702 g) (u + 1);
+// with scale_col >= 0 row t is multiplied by sigmoid(in[t, scale_col]). Rows of `in` are `ld` apart. Eight columns a
+// thread (inter, ld % 8 == 0, 16-byte rows); the grid is (columns, rows).
+template <typename T>
+__global__ void glu_limit8_kernel(const T* __restrict__ in, long long ld, T* __restrict__ out, int rows, int inter, float limit,
+                                  int scale_col) {
+  const int j = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+  if (j >= inter) return;
+  for (int t = blockIdx.y; t < rows; t += gridDim.y) {
+    const T* row = in + (size_t)t * ld;
+    float g[8], u[8];
+    hb::load8(row + j, g);
+    hb::load8(row + inter + j, u);
+    const float s = scale_col >= 0 ? 1.f / (1.f + expf(-hb::to_f32(row[scale_col]))) : 1.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) g[e] = s * hb::clamped_glu(g[e], u[e], limit);
+#pragma unroll
+    for (int e = 0; e < 8; e += 4)
+      store4_any(out, sizeof(T) == 4 ? HB_DTYPE_F32 : HB_DTYPE_BF16, (size_t)t * inter + j + e, make_float4(g[e], g[e + 1], g[e + 2], g[e + 3]));
+  }
+}
+
+template <typename T>
+__global__ void glu_limit_kernel(const T* __restrict__ in, long long ld, T* __restrict__ out, int rows, int inter, float limit,
+                                 int scale_col) {
+  const size_t total = (size_t)rows * inter;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = i / inter;
+    const int j = (int)(i - t * inter);
+    const T* row = in + t * ld;
+    const float s = scale_col >= 0 ? 1.f / (1.f + expf(-hb::to_f32(row[scale_col]))) : 1.f;
+    out[i] = hb::from_f32<T>(s * hb::clamped_glu(hb::to_f32(row[j]), hb::to_f32(row[inter + j]), limit));
+  }
+}
+
+extern "C" int hb_glu_limit(const void* in, long long ld, void* out, int dtype, int rows, int inter, float limit, int scale_col,
+                            cudaStream_t stream) {
+  if (!in || !out || rows < 0 || inter <= 0 || ld < 2 * (long long)inter || scale_col >= ld || !(limit > 0.f) || !dtype_ok(dtype))
+    return HB_ERR_BAD_ARG;
+  if (rows == 0) return HB_OK;
+  if (inter % 8 == 0 && ld % 8 == 0 && ((uintptr_t)in & 15) == 0) {
+    const int threads = inter / 8 >= 256 ? 256 : ((inter / 8 + 31) / 32) * 32;
+    const int cols = (inter / 8 + threads - 1) / threads;
+    int down = 148 * 2048 / (threads * cols);
+    down = rows < down ? rows : (down < 1 ? 1 : down);
+    if (down > 65535) down = 65535;
+    const dim3 grid(cols, down);
+    if (dtype == HB_DTYPE_F32) glu_limit8_kernel<float><<<grid, threads, 0, stream>>>((const float*)in, ld, (float*)out, rows, inter, limit, scale_col);
+    else glu_limit8_kernel<__nv_bfloat16><<<grid, threads, 0, stream>>>((const __nv_bfloat16*)in, ld, (__nv_bfloat16*)out, rows, inter, limit, scale_col);
+  } else {
+    const size_t want = ((size_t)rows * inter + 255) / 256;
+    const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
+    if (dtype == HB_DTYPE_F32) glu_limit_kernel<float><<<blocks, 256, 0, stream>>>((const float*)in, ld, (float*)out, rows, inter, limit, scale_col);
+    else glu_limit_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)in, ld, (__nv_bfloat16*)out, rows, inter, limit, scale_col);
+  }
   HB_LAUNCH_CHECK();
   return HB_OK;
 }

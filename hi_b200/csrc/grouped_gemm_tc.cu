@@ -22,7 +22,8 @@
 //               tokens) and write the epilogue:
 //     DUAL   two weight stacks (gate, up), two accumulators: act = silu(s*g) * (s*u), bfloat16,
 //            where s is the token's router score (crates/hi-mlx/src/models.rs:6086-6100: the score
-//            scales the expert input, which is the same by linearity);
+//            scales the expert input, which is the same by linearity), or with `limit` > 0 the clamped
+//            unit min(g, limit) sigmoid(1.702 .) (clamp(u) + 1);
 //     else   the float32 product (down projection).
 // Tensor memory is two slots of 256 columns. A tile takes one slot, and the next tile
 // accumulates into the other while this one is written out; only a DUAL tile of more than 128
@@ -68,6 +69,7 @@ struct Params {
   int experts, n_out, K, rows;
   float* scratch;            // not DUAL: [blocks of the launch][BT][BF] partial tiles of the last round's pieces, or null
   int* counters;             // [blocks of the launch] pieces of each cut tile that have arrived; zero between launches
+  float limit;               // DUAL: > 0: the clamped unit (hb::clamped_glu) instead of SwiGLU
   int relu2;                 // not DUAL, whole tiles only: out = bfloat16 max(x W^T, 0)^2 (an expert's up stack without a gate)
 };
 constexpr int MAX_PIECES = 4;    // a tile of the last round is cut into at most this many pieces
@@ -312,7 +314,13 @@ grouped_gemm_tc_kernel(const __grid_constant__ Maps maps, const Params p) {
                 const float gs = s * __uint_as_float(g[j + h]);
                 // silu by the fast exponential and division: their error is far below the
                 // bfloat16 rounding of the result
-                a[h] = __fdividef(gs, 1.f + __expf(-gs)) * (s * __uint_as_float(u[j + h]));
+                const float us = s * __uint_as_float(u[j + h]);
+                if (p.limit > 0.f) {
+                  const float gc = fminf(gs, p.limit);
+                  a[h] = __fdividef(gc, 1.f + __expf(-1.702f * gc)) * (fminf(fmaxf(us, -p.limit), p.limit) + 1.f);
+                } else {
+                  a[h] = __fdividef(gs, 1.f + __expf(-gs)) * us;
+                }
               }
               __nv_bfloat162 pr = __floats2bfloat162_rn(a[0], a[1]);
               packed[q][j >> 1] = *reinterpret_cast<uint32_t*>(&pr);
@@ -484,7 +492,7 @@ extern "C" int hb_gather_rows(const void* x, const int* sorted_entry, int top_k,
 // `status` is one int on the device, zero before the call; nonzero afterwards = a wait timed out.
 extern "C" int hb_moe_gate_up_tc(const void* xs, const int* sorted_entry, const void* w_gate, const void* w_up,
                                  const int* offsets, int experts, const float* scores, void* act, int rows, int inter,
-                                 int hidden, int* status, cudaStream_t stream) {
+                                 int hidden, float limit, int* status, cudaStream_t stream) {
   if (!xs || !sorted_entry || !w_gate || !w_up || !offsets || !scores || !act || !status || rows < 0 || experts <= 0)
     return HB_ERR_BAD_ARG;
   if (hidden % 8 != 0 || inter % 8 != 0 || hidden <= 0 || inter <= 0) return HB_ERR_UNSUPPORTED;
@@ -493,7 +501,7 @@ extern "C" int hb_moe_gate_up_tc(const void* xs, const int* sorted_entry, const 
   const int bt = few ? BT_SHORT : BT_LONG;
   const int max_tiles = (rows + bt - 1) / bt + (experts < rows ? experts : rows);
   if (max_tiles > 65535) return HB_ERR_UNSUPPORTED;
-  Params p{offsets, sorted_entry, scores, act, status, experts, inter, hidden, rows, nullptr, nullptr};
+  Params p{offsets, sorted_entry, scores, act, status, experts, inter, hidden, rows, nullptr, nullptr, limit, 0};
   return few ? launch<true, 5, BT_SHORT>(xs, w_gate, w_up, p, max_tiles, stream)
              : launch<true, 4, BT_LONG>(xs, w_gate, w_up, p, max_tiles, stream);
 }
@@ -516,7 +524,7 @@ extern "C" int hb_moe_down_tc(const void* act, const void* w_down, const int* of
   if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess)
     return HB_ERR_BAD_ARG;
   const bool room = scratch && counters && n_counters >= sms && scratch_floats >= (long long)sms * bt * BF;
-  Params p{offsets, nullptr, nullptr, y, status, experts, hidden, inter, rows, room ? scratch : nullptr, counters};
+  Params p{offsets, nullptr, nullptr, y, status, experts, hidden, inter, rows, room ? scratch : nullptr, counters, 0.f, 0};
   return few ? launch<false, 8, BT_SHORT>(act, w_down, nullptr, p, max_tiles, stream)
              : launch<false, 5, BT_LONG>(act, w_down, nullptr, p, max_tiles, stream);
 }
@@ -532,7 +540,7 @@ extern "C" int hb_moe_up_relu2_tc(const void* xs, const void* w_up, const int* o
   const int bt = few ? BT_SHORT : BT_LONG;
   const int max_tiles = (rows + bt - 1) / bt + (experts < rows ? experts : rows);
   if (max_tiles > 65535) return HB_ERR_UNSUPPORTED;
-  Params p{offsets, nullptr, nullptr, act, status, experts, inter, hidden, rows, nullptr, nullptr, 1};
+  Params p{offsets, nullptr, nullptr, act, status, experts, inter, hidden, rows, nullptr, nullptr, 0.f, 1};
   return few ? launch<false, 8, BT_SHORT>(xs, w_up, nullptr, p, max_tiles, stream)
              : launch<false, 5, BT_LONG>(xs, w_up, nullptr, p, max_tiles, stream);
 }

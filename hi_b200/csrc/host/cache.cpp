@@ -40,13 +40,14 @@ int PagePool::give(int page, int64_t owner) {
   return HBH_OK;
 }
 
-CacheManager::CacheManager(int n_groups, const int* window_kind, const int64_t* window_size, const int* pages,
-                           int page_size, int max_requests)
+CacheManager::CacheManager(int n_groups, const int* window_kind, const int64_t* window_size,
+                           const int64_t* window_keep, const int* pages, int page_size, int max_requests)
     : page_size_(page_size), max_requests_(max_requests) {
   for (int g = 0; g < n_groups; ++g) {
     Window w;
     w.kind = window_kind[g];
     w.size = window_size[g];
+    w.keep = window_keep ? window_keep[g] : 0;
     windows_.push_back(w);
     pools_.emplace_back(pages[g]);
   }
@@ -86,15 +87,22 @@ int CacheManager::close(int64_t request) {
   return rc;
 }
 
+// Pages that blocks have .. need_blocks - 1 take: blocks wholly before the window of the token at `length` are
+// never read (unless they hold kept tokens) and get none.
+int64_t CacheManager::new_pages(const Window& w, int64_t have, int64_t length, int64_t need_blocks) const {
+  const int64_t first_live = w.first_live(length) / page_size_;
+  const int64_t live = std::max<int64_t>(0, need_blocks - std::max(have, first_live));
+  const int64_t kept = std::max<int64_t>(0, std::min({w.kept_blocks(page_size_), first_live, need_blocks}) - have);
+  return live + kept;
+}
+
 void CacheManager::pages_needed(int64_t request, int n_new, int64_t length, int* out) {
   const RequestCache* rc = request >= 0 ? find(request) : nullptr;
   if (rc) length = rc->length;
   const int64_t need_blocks = blocks_for(length, n_new);
   for (size_t g = 0; g < windows_.size(); ++g) {
     const int64_t have = rc ? (int64_t)rc->tables[g].size() : 0;
-    // blocks wholly before the window of the first new token are never read
-    const int64_t first_live = windows_[g].first_live(length) / page_size_;
-    out[g] = (int)std::max<int64_t>(0, need_blocks - std::max(have, first_live));
+    out[g] = (int)new_pages(windows_[g], have, length, need_blocks);
   }
 }
 
@@ -104,13 +112,12 @@ void CacheManager::peak_pages_needed(int64_t request, int64_t n_new, int64_t len
   const int64_t need_blocks = (length + n_new + page_size_ - 1) / page_size_;
   for (size_t g = 0; g < windows_.size(); ++g) {
     const int64_t have = rc ? (int64_t)rc->tables[g].size() : 0;
-    const int64_t first_live = windows_[g].first_live(length) / page_size_;
-    int64_t need = std::max<int64_t>(0, need_blocks - std::max(have, first_live));
+    int64_t need = new_pages(windows_[g], have, length, need_blocks);
     if (windows_[g].kind != HBH_WINDOW_NONE) {
       int64_t held = 0;
       if (rc)
         for (int page : rc->tables[g]) held += page != HBH_FREED;
-      const int64_t most = (windows_[g].size + page_size_ - 1) / page_size_ + 1;
+      const int64_t most = windows_[g].most_pages(page_size_);
       need = std::min(need, std::max<int64_t>(0, most - held));
     }
     out[g] = (int)need;
@@ -142,10 +149,11 @@ int CacheManager::reserve(int64_t request, int n_new, int* fail) {
   for (size_t g = 0; g < windows_.size(); ++g) {
     std::vector<int>& table = rc->tables[g];
     const int64_t first_live = windows_[g].first_live(rc->length) / page_size_;
+    const int64_t kept = windows_[g].kept_blocks(page_size_);
     if ((int64_t)table.size() < need_blocks) rc->version = ++versions_;
     while ((int64_t)table.size() < need_blocks) {
       int page = HBH_FREED;
-      if ((int64_t)table.size() >= first_live) {
+      if ((int64_t)table.size() >= first_live || (int64_t)table.size() < kept) {
         const int r = pools_[g].take(request, &page);
         if (r != HBH_OK) return r;      // cannot happen: the need was checked against the pool above
       }
@@ -183,7 +191,7 @@ int CacheManager::commit(int64_t request, int n_new) {
     const int64_t dead_blocks = windows_[g].first_live(rc->length) / page_size_;
     std::vector<int>& table = rc->tables[g];
     const int64_t upto = std::min<int64_t>(dead_blocks, (int64_t)table.size());
-    for (int64_t b = 0; b < upto; ++b)
+    for (int64_t b = windows_[g].kept_blocks(page_size_); b < upto; ++b)
       if (table[b] != HBH_FREED) {
         const int r = pools_[g].give(table[b], request);
         if (r != HBH_OK) return r;
@@ -278,16 +286,17 @@ int64_t hbh_pool_stat(void* pool, int what) {
   return HBH_ERR_ARG;
 }
 
-void* hbh_cache_create(int n_groups, const int* window_kind, const int64_t* window_size, const int* pages,
-                       int page_size, int max_requests) {
+void* hbh_cache_create(int n_groups, const int* window_kind, const int64_t* window_size, const int64_t* window_keep,
+                       const int* pages, int page_size, int max_requests) {
   if (n_groups < 0 || page_size <= 0 || max_requests < 0) return nullptr;
   for (int g = 0; g < n_groups; ++g) {
     if (pages[g] <= 0) return nullptr;
     if (window_kind[g] != HBH_WINDOW_NONE && window_kind[g] != HBH_WINDOW_CHUNK && window_kind[g] != HBH_WINDOW_SLIDING)
       return nullptr;
     if (window_kind[g] != HBH_WINDOW_NONE && window_size[g] <= 0) return nullptr;
+    if (window_keep && (window_keep[g] < 0 || (window_keep[g] > 0 && window_kind[g] != HBH_WINDOW_SLIDING))) return nullptr;
   }
-  return new CacheManager(n_groups, window_kind, window_size, pages, page_size, max_requests);
+  return new CacheManager(n_groups, window_kind, window_size, window_keep, pages, page_size, max_requests);
 }
 void hbh_cache_destroy(void* cache) { delete static_cast<CacheManager*>(cache); }
 const char* hbh_cache_error(void* cache) { return static_cast<CacheManager*>(cache)->error.c_str(); }

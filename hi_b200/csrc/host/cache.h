@@ -36,12 +36,18 @@ class PagePool {
 struct Window {
   int kind = HBH_WINDOW_NONE;
   int64_t size = 0;
+  int64_t keep = 0;                         // sliding windows: the first `keep` tokens stay readable for good
   // oldest position a query at `next_position` or later can still read
   int64_t first_live(int64_t next_position) const {
     if (kind == HBH_WINDOW_CHUNK) return (next_position / size) * size;
     if (kind == HBH_WINDOW_SLIDING) return next_position - size + 1 > 0 ? next_position - size + 1 : 0;
     return 0;
   }
+  // blocks at the start of a request that hold kept tokens: their pages are never given back before it ends
+  int64_t kept_blocks(int64_t page_size) const { return (keep + page_size - 1) / page_size; }
+  // most pages a request holds at a time when its tokens come one by one: the kept ones, the window, the page
+  // being written
+  int64_t most_pages(int64_t page_size) const { return kept_blocks(page_size) + (size + page_size - 1) / page_size + 1; }
 };
 
 struct RequestCache {
@@ -54,8 +60,8 @@ struct RequestCache {
 
 class CacheManager {
  public:
-  CacheManager(int n_groups, const int* window_kind, const int64_t* window_size, const int* pages, int page_size,
-               int max_requests);
+  CacheManager(int n_groups, const int* window_kind, const int64_t* window_size, const int64_t* window_keep, const int* pages,
+               int page_size, int max_requests);
   int n_groups() const { return (int)windows_.size(); }
   int page_size() const { return page_size_; }
   int max_requests() const { return max_requests_; }
@@ -82,6 +88,7 @@ class CacheManager {
   std::string error;
 
  private:
+  int64_t new_pages(const Window& w, int64_t have, int64_t length, int64_t need_blocks) const;
   int64_t blocks_for(int64_t length, int n_new) const { return (length + n_new + page_size_ - 1) / page_size_; }
   int page_size_, max_requests_;
   int64_t versions_ = 0;

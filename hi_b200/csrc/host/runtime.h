@@ -44,8 +44,9 @@ int hbh_pool_owner(void* pool, int page, int64_t* owner, int* held);
 int64_t hbh_pool_stat(void* pool, int what);
 
 // ---- the cache manager
-void* hbh_cache_create(int n_groups, const int* window_kind, const int64_t* window_size, const int* pages,
-                       int page_size, int max_requests);
+// window_keep [n_groups] (or null): sliding windows only, the first tokens of a request that stay readable for good
+void* hbh_cache_create(int n_groups, const int* window_kind, const int64_t* window_size, const int64_t* window_keep,
+                       const int* pages, int page_size, int max_requests);
 void hbh_cache_destroy(void* cache);
 const char* hbh_cache_error(void* cache);
 void* hbh_cache_pool(void* cache, int group);                 // borrowed; lives as long as the cache

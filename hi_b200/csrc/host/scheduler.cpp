@@ -167,8 +167,8 @@ int Scheduler::add(int64_t id, int64_t prompt_len, int64_t max_tokens) {
   for (int g = 0; g < cache_->n_groups(); ++g) {
     int64_t need = (total + ps - 1) / ps;
     const Window& w = cache_->window(g);
-    // a windowed group holds at most its window plus the page being written
-    if (w.kind != HBH_WINDOW_NONE) need = std::min(need, (w.size + ps - 1) / ps + 1);
+    // a windowed group holds at most its kept tokens, its window and the page being written
+    if (w.kind != HBH_WINDOW_NONE) need = std::min(need, w.most_pages(ps));
     if (need > cache_->pool(g).total()) {
       error = "insufficient_gpu_memory: the request needs " + std::to_string(need) + " page(s) of group " +
               std::to_string(g) + ", the pool has " + std::to_string(cache_->pool(g).total());

@@ -226,7 +226,7 @@ constexpr int ROUTER_FEW_EXP = 4;
 
 template <typename TX, typename TW>
 __global__ void __launch_bounds__(ROUTER_FEW_EXP * ROUTER_KPARTS * 32)
-router_few_kernel(const TX* __restrict__ x, const TW* __restrict__ w, int n, int hidden, int experts, int top_k,
+router_few_kernel(const TX* __restrict__ x, const TW* __restrict__ w, const float* __restrict__ bias, int n, int hidden, int experts, int top_k,
                   int mode, float score_scale, float* logits, int* ids, float* scores, int* __restrict__ offsets,
                   int* __restrict__ sorted_entry, int* __restrict__ slot_of_entry, int* __restrict__ active,
                   int* counter) {
@@ -280,7 +280,7 @@ router_few_kernel(const TX* __restrict__ x, const TW* __restrict__ w, int n, int
       float total = partial[threadIdx.x][0];
 #pragma unroll
       for (int q = 1; q < ROUTER_KPARTS; ++q) total += partial[threadIdx.x][q];
-      logits[(size_t)t * experts + mine] = total;
+      logits[(size_t)t * experts + mine] = bias ? total + bias[mine] : total;
     }
     __threadfence();
   }
@@ -316,7 +316,7 @@ constexpr int ROUTER_TOK = 4, ROUTER_EXP = 16;
 
 template <typename TW>
 __global__ void __launch_bounds__(ROUTER_KPARTS * 32)
-router_logits_tiled_kernel(const float* __restrict__ x, const TW* __restrict__ w, int n, int hidden, int experts,
+router_logits_tiled_kernel(const float* __restrict__ x, const TW* __restrict__ w, const float* __restrict__ bias, int n, int hidden, int experts,
                            int top_k, int mode, float score_scale, float* __restrict__ logits, int* __restrict__ ids,
                            float* __restrict__ scores) {
   __shared__ float partial[ROUTER_KPARTS][ROUTER_TOK][ROUTER_EXP];
@@ -379,6 +379,7 @@ router_logits_tiled_kernel(const float* __restrict__ x, const TW* __restrict__ w
     float total = partial[0][tt][e];
 #pragma unroll
     for (int q = 1; q < ROUTER_KPARTS; ++q) total += partial[q][tt][e];
+    if (bias && e0 + e < experts) total += bias[e0 + e];
     lg[tt][e] = total;
     if (logits && t0 + tt < n && e0 + e < experts) logits[(size_t)(t0 + tt) * experts + e0 + e] = total;
   }
@@ -422,6 +423,7 @@ int launch_plan(const int* ids, int n, int experts, int* offsets, int* sorted_en
 // ------------------------------------------------------------------ grouped products, general form
 // C[r, n] = sum_k A[row(r), k] * W[e(r), n, k] for the sorted slots r of every expert e.
 // MODE 1 (DUAL): two weight stacks (gate, up); out = silu(s*g) * (s*u) in the engine dtype.
+//         with limit > 0 the epilogue is the clamped unit instead (hb::clamped_glu).
 // MODE 2: one stack; out = max(s*u, 0)^2 in the engine dtype (an expert without a gate branch).
 // MODE 0: out = float32 product (the down projection).
 // Tiles BM x BN over (expert, rows of that expert) x columns; any K, any number of columns.
@@ -432,7 +434,7 @@ __global__ void grouped_gemm_kernel(const T* __restrict__ A, int lda, const int*
                                     int top_k, const T* __restrict__ W0, const T* __restrict__ W1,
                                     const int* __restrict__ offsets, int experts,
                                     const float* __restrict__ scores, void* __restrict__ out, int n_out,
-                                    int K) {
+                                    int K, float limit) {
   constexpr bool DUAL = MODE == 1;
   __shared__ float As[BK][BM + 1];
   __shared__ float Bs0[BK][BN + 1];
@@ -515,7 +517,7 @@ __global__ void grouped_gemm_kernel(const T* __restrict__ A, int lda, const int*
       if (n >= n_out) continue;
       if (DUAL) {
         const float g = s * acc0[rr][c], u = s * acc1[rr][c];
-        reinterpret_cast<T*>(out)[(size_t)slot * n_out + n] = hb::from_f32<T>(g / (1.f + expf(-g)) * u);
+        reinterpret_cast<T*>(out)[(size_t)slot * n_out + n] = hb::from_f32<T>(limit > 0.f ? hb::clamped_glu(g, u, limit) : g / (1.f + expf(-g)) * u);
       } else if (MODE == 2) {
         const float u = fmaxf(s * acc0[rr][c], 0.f);
         reinterpret_cast<T*>(out)[(size_t)slot * n_out + n] = hb::from_f32<T>(u * u);
@@ -537,7 +539,7 @@ template <typename T, int MODE, int R>
 __device__ __forceinline__ void gemv_rows(const T* __restrict__ A, int lda, const int* __restrict__ sorted_entry,
                                           int top_k, const T* __restrict__ w0, const T* __restrict__ w1,
                                           const float* __restrict__ scores, void* __restrict__ out, int n_out,
-                                          int K, int n, int r0, int lane) {
+                                          int K, int n, int r0, int lane, float limit) {
   // gate/up streams two weight rows per lane; the down projection has one, and needs twice the
   // unroll for as many bytes in flight (measured at three blocks per SM: 4 and 8 beat 2, 3 or 8 and 4 or 16)
   constexpr bool DUAL = MODE == 1;
@@ -591,7 +593,7 @@ __device__ __forceinline__ void gemv_rows(const T* __restrict__ A, int lda, cons
       const size_t o = (size_t)(r0 + r) * n_out + n;
       if (DUAL) {
         const float gg = sc[r] * gs, uu = sc[r] * us;
-        reinterpret_cast<T*>(out)[o] = hb::from_f32<T>(gg / (1.f + expf(-gg)) * uu);
+        reinterpret_cast<T*>(out)[o] = hb::from_f32<T>(limit > 0.f ? hb::clamped_glu(gg, uu, limit) : gg / (1.f + expf(-gg)) * uu);
       } else if (MODE == 2) {
         const float uu = fmaxf(sc[r] * gs, 0.f);
         reinterpret_cast<T*>(out)[o] = hb::from_f32<T>(uu * uu);
@@ -607,7 +609,7 @@ __global__ void __launch_bounds__(GEMV_WARPS * 32, 3)   // three blocks per SM (
 grouped_gemv_kernel(const T* __restrict__ A, int lda, const int* __restrict__ sorted_entry, int top_k,
                     const T* __restrict__ W0, const T* __restrict__ W1, const int* __restrict__ offsets,
                     const int* __restrict__ active, const float* __restrict__ scores, void* __restrict__ out,
-                    int n_out, int K) {
+                    int n_out, int K, float limit) {
   // blockIdx.y counts the experts that have rows; the grid has min(experts, entries) of them
   if ((int)blockIdx.y >= active[0]) return;
   const int e = active[1 + blockIdx.y];
@@ -622,32 +624,32 @@ grouped_gemv_kernel(const T* __restrict__ A, int lda, const int* __restrict__ so
   // rows in runs of 8, 4, 2, 1: every row count is covered, each weight element is reused by
   // the whole run
   for (; r0 + 8 <= end; r0 += 8)
-    gemv_rows<T, MODE, 8>(A, lda, sorted_entry, top_k, w0, w1, scores, out, n_out, K, n, r0, lane);
+    gemv_rows<T, MODE, 8>(A, lda, sorted_entry, top_k, w0, w1, scores, out, n_out, K, n, r0, lane, limit);
   if (r0 + 4 <= end) {
-    gemv_rows<T, MODE, 4>(A, lda, sorted_entry, top_k, w0, w1, scores, out, n_out, K, n, r0, lane);
+    gemv_rows<T, MODE, 4>(A, lda, sorted_entry, top_k, w0, w1, scores, out, n_out, K, n, r0, lane, limit);
     r0 += 4;
   }
   if (r0 + 2 <= end) {
-    gemv_rows<T, MODE, 2>(A, lda, sorted_entry, top_k, w0, w1, scores, out, n_out, K, n, r0, lane);
+    gemv_rows<T, MODE, 2>(A, lda, sorted_entry, top_k, w0, w1, scores, out, n_out, K, n, r0, lane, limit);
     r0 += 2;
   }
-  if (r0 < end) gemv_rows<T, MODE, 1>(A, lda, sorted_entry, top_k, w0, w1, scores, out, n_out, K, n, r0, lane);
+  if (r0 < end) gemv_rows<T, MODE, 1>(A, lda, sorted_entry, top_k, w0, w1, scores, out, n_out, K, n, r0, lane, limit);
 }
 
 template <typename T, int MODE>
 int launch_grouped_mode(const void* A, int lda, const int* sorted_entry, int top_k, const void* W0, const void* W1,
                         const int* offsets, const int* active, int experts, const float* scores, void* out,
-                        int n_entries, int n_out, int K, int few_rows, cudaStream_t stream) {
+                        int n_entries, int n_out, int K, int few_rows, float limit, cudaStream_t stream) {
   if (few_rows && K % 8 == 0 && lda % 8 == 0) {
     dim3 grid((n_out + GEMV_WARPS - 1) / GEMV_WARPS, experts < n_entries ? experts : n_entries);
     grouped_gemv_kernel<T, MODE><<<grid, GEMV_WARPS * 32, 0, stream>>>(
-        (const T*)A, lda, sorted_entry, top_k, (const T*)W0, (const T*)W1, offsets, active, scores, out, n_out, K);
+        (const T*)A, lda, sorted_entry, top_k, (const T*)W0, (const T*)W1, offsets, active, scores, out, n_out, K, limit);
   } else {
     const int max_tiles = (n_entries + BM - 1) / BM + (experts < n_entries ? experts : n_entries);
     dim3 grid((n_out + BN - 1) / BN, max_tiles);
     if (grid.y > 65535) return HB_ERR_UNSUPPORTED;
     grouped_gemm_kernel<T, MODE><<<grid, GT, 0, stream>>>((const T*)A, lda, sorted_entry, top_k, (const T*)W0,
-                                                          (const T*)W1, offsets, experts, scores, out, n_out, K);
+                                                          (const T*)W1, offsets, experts, scores, out, n_out, K, limit);
   }
   HB_LAUNCH_CHECK();
   return HB_OK;
@@ -657,10 +659,10 @@ int launch_grouped_mode(const void* A, int lda, const int* sorted_entry, int top
 template <typename T>
 int launch_grouped(int mode, const void* A, int lda, const int* sorted_entry, int top_k, const void* W0,
                    const void* W1, const int* offsets, const int* active, int experts, const float* scores, void* out,
-                   int n_entries, int n_out, int K, int few_rows, cudaStream_t stream) {
+                   int n_entries, int n_out, int K, int few_rows, float limit, cudaStream_t stream) {
 #define HB_GROUPED(M)                                                                                              \
   launch_grouped_mode<T, M>(A, lda, sorted_entry, top_k, W0, M == 1 ? W1 : nullptr, offsets, active, experts, scores, \
-                            out, n_entries, n_out, K, few_rows, stream)
+                            out, n_entries, n_out, K, few_rows, limit, stream)
   if (mode == 1) return HB_GROUPED(1);
   if (mode == 2) return HB_GROUPED(2);
   return HB_GROUPED(0);
@@ -673,7 +675,7 @@ namespace {
 
 // The router, and with `counter` (an int that is zero between launches) the plan as well: in the
 // same kernel when a block takes one token, by the plan's own kernel after the tiled one.
-int router_launch(const void* x, int x_dtype, const void* w, int w_dtype, int n, int hidden, int experts, int top_k, int mode,
+int router_launch(const void* x, int x_dtype, const void* w, int w_dtype, const float* bias, int n, int hidden, int experts, int top_k, int mode,
                   float score_scale, float* logits_out, int* ids, float* scores, int* offsets, int* sorted_entry, int* slot_of_entry,
                   int* active, int* counter, cudaStream_t stream) {
   if (!x || !w || !ids || !scores || n < 0 || hidden <= 0 || experts <= 0 || top_k <= 0 || top_k > experts || mode < 0 ||
@@ -696,10 +698,10 @@ int router_launch(const void* x, int x_dtype, const void* w, int w_dtype, int n,
     if (grid.y > 65535) return HB_ERR_UNSUPPORTED;
     if (w_dtype == HB_DTYPE_F32)
       router_logits_tiled_kernel<float><<<grid, ROUTER_KPARTS * 32, 0, stream>>>(
-          (const float*)x, (const float*)w, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores);
+          (const float*)x, (const float*)w, bias, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores);
     else
       router_logits_tiled_kernel<__nv_bfloat16><<<grid, ROUTER_KPARTS * 32, 0, stream>>>(
-          (const float*)x, (const __nv_bfloat16*)w, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores);
+          (const float*)x, (const __nv_bfloat16*)w, bias, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores);
     HB_LAUNCH_CHECK();
     if (grid.y > 1) {
       router_select_kernel<<<(n + 127) / 128, 128, 0, stream>>>(logits_out, n, experts, top_k, mode, score_scale, ids, scores);
@@ -722,15 +724,15 @@ int router_launch(const void* x, int x_dtype, const void* w, int w_dtype, int n,
   const dim3 grid(n, columns);
   if (x_dtype == HB_DTYPE_F32 && w_dtype == HB_DTYPE_F32)
     router_few_kernel<float, float><<<grid, threads, smem, stream>>>(
-        (const float*)x, (const float*)w, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores, offsets,
+        (const float*)x, (const float*)w, bias, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores, offsets,
         sorted_entry, slot_of_entry, active, fused);
   else if (x_dtype == HB_DTYPE_F32 && w_dtype == HB_DTYPE_BF16)
     router_few_kernel<float, __nv_bfloat16><<<grid, threads, smem, stream>>>(
-        (const float*)x, (const __nv_bfloat16*)w, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores,
+        (const float*)x, (const __nv_bfloat16*)w, bias, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores,
         offsets, sorted_entry, slot_of_entry, active, fused);
   else if (x_dtype == HB_DTYPE_BF16 && w_dtype == HB_DTYPE_BF16)
     router_few_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, threads, smem, stream>>>(
-        (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores,
+        (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, bias, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores,
         offsets, sorted_entry, slot_of_entry, active, fused);
   else
     return HB_ERR_BAD_ARG;
@@ -747,15 +749,16 @@ int router_launch(const void* x, int x_dtype, const void* w, int w_dtype, int n,
 
 }  // namespace
 
-extern "C" int hb_router_topk(const void* x, int x_dtype, const void* w, int w_dtype, int n, int hidden,
+// `bias` (float32 [experts] or null) is added to the logits before anything reads them
+extern "C" int hb_router_topk(const void* x, int x_dtype, const void* w, int w_dtype, const float* bias, int n, int hidden,
                               int experts, int top_k, int mode, float score_scale, float* logits_out, int* ids,
                               float* scores, cudaStream_t stream) {
-  return router_launch(x, x_dtype, w, w_dtype, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores, nullptr, nullptr,
+  return router_launch(x, x_dtype, w, w_dtype, bias, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores, nullptr, nullptr,
                        nullptr, nullptr, nullptr, stream);
 }
 
 // Router and plan in one call; `counter` is one int that the caller zeroed once and then leaves alone.
-extern "C" int hb_router_plan(const void* x, int x_dtype, const void* w, int w_dtype, int n, int hidden, int experts,
+extern "C" int hb_router_plan(const void* x, int x_dtype, const void* w, int w_dtype, const float* bias, int n, int hidden, int experts,
                               int top_k, int mode, float score_scale, float* logits_out, int* ids, float* scores,
                               int* offsets, int* sorted_entry, int* slot_of_entry, int* active, int* counter,
                               cudaStream_t stream) {
@@ -764,7 +767,7 @@ extern "C" int hb_router_plan(const void* x, int x_dtype, const void* w, int w_d
   if (n == 0) {  // nothing routed: an empty plan
     return launch_plan(ids, 0, experts, offsets, sorted_entry, slot_of_entry, active, stream);
   }
-  return router_launch(x, x_dtype, w, w_dtype, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores,
+  return router_launch(x, x_dtype, w, w_dtype, bias, n, hidden, experts, top_k, mode, score_scale, logits_out, ids, scores,
                        offsets, sorted_entry, slot_of_entry, active, counter, stream);
 }
 
@@ -777,12 +780,12 @@ extern "C" int hb_moe_plan(const int* ids, int n_entries, int experts, int* offs
 }
 
 // gate/up with SwiGLU: act[slot, :] (engine dtype, [n_entries, inter]). activation 1: experts without a gate
-// branch, act = max(s * x Wu^T, 0)^2 (w_gate is not read).
+// branch, act = max(s * x Wu^T, 0)^2 (w_gate is not read). activation 2: gate/up with the clamped unit of `limit` > 0.
 extern "C" int hb_moe_gate_up(const void* x, int dtype, const int* sorted_entry, int top_k, const void* w_gate,
                               const void* w_up, const int* offsets, const int* active, int experts,
                               const float* scores, void* act, int n_entries, int inter, int hidden, int few_rows,
-                              int activation, cudaStream_t stream) {
-  if (activation != 0 && activation != 1) return HB_ERR_BAD_ARG;
+                              int activation, float limit, cudaStream_t stream) {
+  if (activation < 0 || activation > 2 || (activation == 2) != (limit > 0.f)) return HB_ERR_BAD_ARG;
   if (activation == 1) w_gate = w_up;
   const int mode = activation == 1 ? 2 : 1;
   if (!x || !sorted_entry || !w_gate || !w_up || !offsets || !active || !scores || !act || n_entries < 0 || inter <= 0 ||
@@ -791,10 +794,10 @@ extern "C" int hb_moe_gate_up(const void* x, int dtype, const int* sorted_entry,
   if (n_entries == 0) return HB_OK;
   if (dtype == HB_DTYPE_F32)
     return launch_grouped<float>(mode, x, hidden, sorted_entry, top_k, mode == 2 ? w_up : w_gate, w_up, offsets, active,
-                                 experts, scores, act, n_entries, inter, hidden, few_rows, stream);
+                                 experts, scores, act, n_entries, inter, hidden, few_rows, limit, stream);
   if (dtype == HB_DTYPE_BF16)
     return launch_grouped<__nv_bfloat16>(mode, x, hidden, sorted_entry, top_k, mode == 2 ? w_up : w_gate, w_up, offsets,
-                                         active, experts, scores, act, n_entries, inter, hidden, few_rows, stream);
+                                         active, experts, scores, act, n_entries, inter, hidden, few_rows, limit, stream);
   return HB_ERR_BAD_ARG;
 }
 
@@ -807,9 +810,9 @@ extern "C" int hb_moe_down(const void* act, int dtype, const void* w_down, const
   if (n_entries == 0) return HB_OK;
   if (dtype == HB_DTYPE_F32)
     return launch_grouped<float>(0, act, inter, nullptr, 1, w_down, nullptr, offsets, active, experts, nullptr, y,
-                                 n_entries, hidden, inter, few_rows, stream);
+                                 n_entries, hidden, inter, few_rows, 0.f, stream);
   if (dtype == HB_DTYPE_BF16)
     return launch_grouped<__nv_bfloat16>(0, act, inter, nullptr, 1, w_down, nullptr, offsets, active, experts, nullptr, y,
-                                         n_entries, hidden, inter, few_rows, stream);
+                                         n_entries, hidden, inter, few_rows, 0.f, stream);
   return HB_ERR_BAD_ARG;
 }

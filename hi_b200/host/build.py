@@ -82,7 +82,7 @@ I, L, P = ctypes.c_int, ctypes.c_int64, ctypes.c_void_p
 _SIGNATURES = {
     "hbh_pool_create": (P, [I]), "hbh_pool_destroy": (None, [P]), "hbh_pool_take": (I, [P, L, P]),
     "hbh_pool_give": (I, [P, I, L]), "hbh_pool_owner": (I, [P, I, P, P]), "hbh_pool_stat": (L, [P, I]),
-    "hbh_cache_create": (P, [I, P, P, P, I, I]), "hbh_cache_destroy": (None, [P]),
+    "hbh_cache_create": (P, [I, P, P, P, P, I, I]), "hbh_cache_destroy": (None, [P]),
     "hbh_cache_error": (ctypes.c_char_p, [P]), "hbh_cache_pool": (P, [P, I]), "hbh_cache_open": (I, [P, L, P]),
     "hbh_cache_close": (I, [P, L]), "hbh_cache_is_open": (I, [P, L]), "hbh_cache_free_slots": (I, [P]),
     "hbh_cache_open_requests": (I, [P, P, I]), "hbh_cache_request_stat": (L, [P, L, I]),

@@ -21,30 +21,39 @@ _SIGNATURES = {
     "hb_embed_gather": [P, I, P, P, I, I, I, F, P],
     "hb_add_rmsnorm": [P, P, I, P, I, P, P, P, I, P, I, P, I, P, P, I, I, F, F, I, P],
     "hb_swiglu": [P, P, I, I, I, P],
+    "hb_embed_position": [P, I, P, P, P, P, I, I, I, F, P],
+    "hb_gelu": [P, P, I, c_longlong, P],
+    "hb_glu_limit": [P, c_longlong, P, I, I, I, F, I, P],
+    "hb_diff_prefill_tc": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, F, F, F, I, P, c_longlong, P, P],
+    "hb_diff_merge": [P, P, P, P, c_longlong, P, I, I, I, I, I, I, F, F, F, P],
+    "hb_gate_rows": [P, c_longlong, P, c_longlong, P, I, c_longlong, I, I, I, P],
+    "hb_conv_qkv": [P, I, c_longlong, P, I, P, c_longlong, c_longlong, I, F, P, P, P, I, I, F, P, P, P, P, P, I, P, P, P, I, I,
+                    I, I, I, I, I, I, I, I, P, P],
+    "hb_sandwich_step": [P, P, I, P, I, P, P, P, I, P, F, P, F, P, I, P, P, I, I, P],
     "hb_relu2": [P, I, P, I, c_longlong, P],
     "hb_softcap": [P, F, c_longlong, P],
     "hb_convert": [P, I, P, I, c_longlong, P],
     "hb_moe_combine": [P, P, P, P, I, P, I, I, I, P],
     "hb_qkv_post": [P, I, P, I, I, I, F, I, F, F, P, P, I, I, F, P, I, I, P, P, P, I, P, P, P, I, I, I, I, I, I, P],
-    "hb_paged_attention": [P, I, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, I, F, P, P, I, I, P, P, P],
+    "hb_paged_attention": [P, I, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, F, P, P, I, I, P, P, P],
     "hb_attention_merge": [P, P, P, I, I, I, I, I, I, P, P],
-    "hb_attention_decode": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, I, P, F, P, P, I, I, P, P, P],
+    "hb_attention_decode": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, P, F, P, P, I, I, P, P, P],
     "hb_attention_decode_tma": [P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, F, I, I, I, P, P, P, P],
     "hb_attention_decode_fused": [P, P, I, I, I, F, I, F, F, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, F, I, I, P, P, P, P, P, P, I, F, I, P],
     "hb_attention_prefill": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P],
-    "hb_attention_prefill_reshaped": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, I, F, P, P, P],
+    "hb_attention_prefill_reshaped": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, F, P, P, P, P, P],
     "hb_attention_prefill_tc": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, I, P, I, P, P, P, P],
-    "hb_attention_prefill_tc_reshaped": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, I, F, P, P, I, P, P, P,
+    "hb_attention_prefill_tc_reshaped": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, I, F, P, P, I, P, P, P,
                                          P],
     "hb_sigmoid_prefill_tc": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, P, I, I, P, P],
     "hb_sigmoid_merge": [P, P, P, I, I, P, I, I, I, I, I, P],
-    "hb_router_topk": [P, I, P, I, I, I, I, I, I, F, P, P, P, P],
+    "hb_router_topk": [P, I, P, I, P, I, I, I, I, I, F, P, P, P, P],
     "hb_moe_plan": [P, I, I, P, P, P, P, P],
-    "hb_router_plan": [P, I, P, I, I, I, I, I, I, F, P, P, P, P, P, P, P, P, P],
-    "hb_moe_gate_up": [P, I, P, I, P, P, P, P, I, P, P, I, I, I, I, I, P],
+    "hb_router_plan": [P, I, P, I, P, I, I, I, I, I, F, P, P, P, P, P, P, P, P, P],
+    "hb_moe_gate_up": [P, I, P, I, P, P, P, P, I, P, P, I, I, I, I, I, F, P],
     "hb_moe_down": [P, I, P, P, P, I, P, I, I, I, I, P],
     "hb_gather_rows": [P, P, I, P, I, I, P],
-    "hb_moe_gate_up_tc": [P, P, P, P, P, I, P, P, I, I, I, P, P],
+    "hb_moe_gate_up_tc": [P, P, P, P, P, I, P, P, I, I, I, F, P, P],
     "hb_moe_down_tc": [P, P, P, I, P, I, I, I, P, c_longlong, P, I, P, P],
     "hb_moe_up_relu2_tc": [P, P, P, I, P, I, I, I, P, P],
     "hb_argmax_rows": [P, I, I, I, P, P, P, P, P],
@@ -241,6 +250,41 @@ def swiglu(gate_up: torch.Tensor) -> torch.Tensor:
         raise KernelError("swiglu input needs an even number of columns")
     out = torch.empty((n, two_i // 2), dtype=gate_up.dtype, device=gate_up.device)
     _check(lib().hb_swiglu(_ptr(gate_up), _ptr(out), _dt(gate_up), n, two_i // 2, _stream()), "swiglu")
+    return out
+
+
+def embed_position(table: torch.Tensor, tokens: torch.Tensor, positions: torch.Tensor, turns: torch.Tensor,
+                   scale: float = 1.0) -> torch.Tensor:
+    """:func:`embed_gather` plus a sinusoidal vector of the token's position: entry 2i is sin(2 pi p turns[i]), entry
+    2i + 1 its cosine; ``turns`` (float64 [ceil(H / 2)]) are the frequencies in turns per position."""
+    _need(table, "table"); _need(tokens, "tokens", torch.int32); _need(positions, "positions", torch.int32)
+    _need(turns, "turns", torch.float64)
+    n, (vocab, hidden) = tokens.numel(), table.shape
+    if positions.numel() != n or turns.numel() != (hidden + 1) // 2:
+        raise KernelError("one position per token and one frequency per pair of columns")
+    out = torch.empty((n, hidden), dtype=torch.float32, device=table.device)
+    _check(lib().hb_embed_position(_ptr(table), _dt(table), _ptr(tokens), _ptr(positions), _ptr(turns), _ptr(out), n, hidden,
+                                   vocab, float(scale), _stream()), "embed_position")
+    return out
+
+
+def gelu(x: torch.Tensor) -> torch.Tensor:
+    """0.5 x (1 + erf(x / sqrt 2)), float32 math, same dtype."""
+    _need(x, "x")
+    out = torch.empty_like(x)
+    _check(lib().hb_gelu(_ptr(x), _ptr(out), _dt(x), x.numel(), _stream()), "gelu")
+    return out
+
+
+def glu_limit(x: torch.Tensor, inter: int, limit: float, scale_col: int = -1) -> torch.Tensor:
+    """Rows [gate (I) | up (I) | ...] -> min(gate, limit) sigmoid(1.702 min(gate, limit)) (clamp(up, +-limit) + 1),
+    [N, I], same dtype, float32 math; with ``scale_col`` >= 0 row t is multiplied by sigmoid(x[t, scale_col])."""
+    _need(x, "x")
+    n, width = x.shape
+    if width < 2 * inter or scale_col >= width:
+        raise KernelError("the rows are too short for gate and up")
+    out = torch.empty((n, inter), dtype=x.dtype, device=x.device)
+    _check(lib().hb_glu_limit(_ptr(x), width, _ptr(out), _dt(x), n, inter, float(limit), int(scale_col), _stream()), "glu_limit")
     return out
 
 
@@ -925,8 +969,13 @@ DECODE_RESIDENT_BLOCKS = 148 * 3   # blocks of the decode kernel resident at a t
 def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
                     seq_of_token: torch.Tensor, positions: torch.Tensor, chunk: int, window: int,
                     scale: float, max_context: int = 0, sink: bool = False, softcap: float = 0.0,
-                    slopes: Optional[torch.Tensor] = None, sink_values: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    slopes: Optional[torch.Tensor] = None, sink_values: Optional[torch.Tensor] = None,
+                    keep: int = 0, parts: bool = False):
     """softmax(q k^T * scale) v over the keys each token may read; q [N, nh, hd] -> [N, nh, hd].
+    ``keep`` (with a sliding ``window``): the first ``keep`` positions stay readable although the window has passed
+    them. ``parts`` (here, in :func:`decode_attention` and :func:`prefill_attention`): the result is not merged;
+    returns ``(part_acc [N, nh, splits, hd], part_ml [N, nh, splits, 2])`` float32, the splits' unnormalised rows with
+    their (max, sum), for :func:`diff_merge`.
     ``sink`` (here and in the other attention kernels): the softmax's denominator has one more term of
     score 0, p_j = e^{s_j} / (1 + sum_j e^{s_j}); the term has no value. ``sink_values`` (float32 [nh]): the
     term's score is the head's own number instead of 0. ``softcap`` > 0: the scaled score becomes
@@ -952,24 +1001,24 @@ def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
             _need(t, nm, torch.float32)
             if t.numel() != nh:
                 raise KernelError(f"{nm} needs one number per query head")
-    out = torch.empty_like(q)
+    out = None if parts else torch.empty_like(q)
     longest = max_context
     if chunk > 0:
         longest = min(longest, chunk)
     if window > 0:
-        longest = min(longest, window)
+        longest = min(longest, window + keep)
     splits = max(1, -(-longest // ATTENTION_SPLIT))
     part_acc = part_ml = None
-    if splits > 1:
+    if splits > 1 or parts:
         part_acc = torch.empty((n, nh, splits, hd), dtype=torch.float32, device=q.device)
         part_ml = torch.empty((n, nh, splits, 2), dtype=torch.float32, device=q.device)
     _check(lib().hb_paged_attention(_ptr(q), _dt(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
                                     block_table.shape[1], _ptr(seq_of_token), _ptr(positions), _ptr(out), n, nh, nkv,
-                                    hd, page_size, int(chunk), int(window), float(scale),
+                                    hd, page_size, int(chunk), int(window), int(keep), float(scale),
                                     int(sink or sink_values is not None), float(softcap), _ptr(slopes),
                                     _ptr(sink_values), ATTENTION_SPLIT, splits, _ptr(part_acc), _ptr(part_ml), _stream()),
            "paged_attention")
-    return out
+    return (part_acc, part_ml) if parts else out
 
 
 def sigmoid_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
@@ -1063,7 +1112,7 @@ def sigmoid_decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: to
     part_acc = torch.empty((n, nh, splits, hd), dtype=torch.float32, device=q.device)
     _check(lib().hb_attention_decode(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
                                      _ptr(seq_of_token), _ptr(positions), _ptr(part_acc), n, nh, nkv, hd, page_size,
-                                     int(chunk), int(window), float(scale), 2, _ptr(head_bias), 0.0, None, None, split_size,
+                                     int(chunk), int(window), 0, float(scale), 2, _ptr(head_bias), 0.0, None, None, split_size,
                                      splits, _ptr(part_acc), None, _stream()), "attention_decode")
     return sigmoid_merge(part_acc, positions, q.dtype, v_inv_freq, v_interleaved)
 
@@ -1136,15 +1185,17 @@ def _decode_splits(longest: int, groups: int) -> Tuple[int, int]:
 TC_ROW_LENGTHS = (64, 128, 192)
 
 
-def decode_attention_supported(q_dtype: torch.dtype, nh: int, nkv: int, hd: int) -> bool:
-    """Shapes the tensor-core decode kernel takes; anything else goes to the general kernel."""
-    return q_dtype == torch.bfloat16 and hd in TC_ROW_LENGTHS and nh % nkv == 0 and nh // nkv <= 16
+def decode_attention_supported(q_dtype: torch.dtype, nh: int, nkv: int, hd: int, row_tiles: bool = False) -> bool:
+    """Shapes the tensor-core decode kernel takes; anything else goes to the general kernel. ``row_tiles``: more
+    than 16 query heads on a kv head are taken in tiles of 16 (by the kernel that loads its tiles by cp.async)."""
+    return q_dtype == torch.bfloat16 and hd in TC_ROW_LENGTHS and nh % nkv == 0 and (row_tiles or nh // nkv <= 16)
 
 
 def decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
                      seq_of_token: torch.Tensor, positions: torch.Tensor, chunk: int, window: int, scale: float,
                      max_context: int, sink: bool = False, softcap: float = 0.0,
-                     slopes: Optional[torch.Tensor] = None, sink_values: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     slopes: Optional[torch.Tensor] = None, sink_values: Optional[torch.Tensor] = None,
+                     keep: int = 0, parts: bool = False):
     """Attention for a batch of single decoded tokens (every row of ``q`` is one request's
     token), bfloat16, split over runs of ``ATTENTION_SPLIT`` keys. Uses scratch memory for the
     partial results of the splits. ``softcap``, ``slopes``, ``sink_values``: as :func:`paged_attention`
@@ -1156,20 +1207,22 @@ def decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
     _, nkv, page_size, hd2 = k_pages.shape
     if hd2 != hd or k_pages.shape != v_pages.shape:
         raise KernelError("cache pages do not match the query's head_dim")
-    if not decode_attention_supported(q.dtype, nh, nkv, hd):
+    if not decode_attention_supported(q.dtype, nh, nkv, hd, row_tiles=parts):
         raise KernelError(f"decode attention does not take nh={nh} nkv={nkv} head_dim={hd}")
     longest = max(int(max_context), 1)
     if chunk > 0:
         longest = min(longest, chunk)
-    if window > 0:
+    if window > 0 and keep > 0:      # walked in tiles of 64 positions: the window's (one more where it straddles), the kept tokens'
+        longest = min(-(-longest // 64), -(-(window + 63) // 64) + -(-keep // 64)) * 64
+    elif window > 0:
         longest = min(longest, window)
-    split_size, splits = _decode_splits(longest, n * nkv)
-    out = torch.empty_like(q)
+    split_size, splits = _decode_splits(longest, n * nkv * -(-(nh // nkv) // 16))
+    out = None if parts else torch.empty_like(q)
     part_acc = part_ml = None
-    if splits > 1:
+    if splits > 1 or parts:
         part_acc = torch.empty((n, nh, splits, hd), dtype=torch.float32, device=q.device)
         part_ml = torch.empty((n, nh, splits, 2), dtype=torch.float32, device=q.device)
-    reshaped = bool(softcap) or slopes is not None or sink_values is not None
+    reshaped = bool(softcap) or slopes is not None or sink_values is not None or keep > 0 or parts
     for t, nm in ((slopes, "slopes"), (sink_values, "sink_values")):
         if t is not None:
             _need(t, nm, torch.float32)
@@ -1184,13 +1237,15 @@ def decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
     if code == _UNSUPPORTED:
         code = lib().hb_attention_decode(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
                                          _ptr(seq_of_token), _ptr(positions), _ptr(out), n, nh, nkv, hd, page_size,
-                                         int(chunk), int(window), float(scale), int(sink), None, float(softcap),
+                                         int(chunk), int(window), int(keep), float(scale), int(sink), None, float(softcap),
                                          _ptr(slopes), _ptr(sink_values), split_size, splits,
                                          _ptr(part_acc), _ptr(part_ml), _stream())
         _check(code, "attention_decode")
     else:
         TC_USED[0] = True
         _check(code, "attention_decode_tma")
+    if parts:
+        return part_acc, part_ml
     if splits > 1:
         _check(lib().hb_attention_merge(_ptr(part_acc), _ptr(part_ml), _ptr(out), _dt(out), n * nh, hd, splits,
                                         int(sink), nh, _ptr(sink_values), _stream()), "attention_merge")
@@ -1283,12 +1338,13 @@ def prefill_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
                       cu_seqlens: torch.Tensor, positions: torch.Tensor, n_seqs: int, max_new: int, chunk: int,
                       window: int, scale: float, skip_single: bool = False,
                       out: Optional[torch.Tensor] = None, sink: bool = False, softcap: float = 0.0,
-                      slopes: Optional[torch.Tensor] = None, sink_values: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      slopes: Optional[torch.Tensor] = None, sink_values: Optional[torch.Tensor] = None,
+                      keep: int = 0, parts: bool = False):
     """Attention for portions of prompts: request ``s`` owns rows ``cu_seqlens[s]..cu_seqlens[s+1]``
     of ``q`` [N, nh, hd], at consecutive positions; bfloat16, flash attention on tensor cores.
     ``skip_single`` leaves the rows of requests that bring one token unwritten (the caller runs
-    the decode kernel for them and passes the same ``out``). ``softcap``, ``slopes``, ``sink_values``: as
-    :func:`paged_attention`."""
+    the decode kernel for them and passes the same ``out``). ``softcap``, ``slopes``, ``sink_values``, ``keep``,
+    ``parts`` (one split): as :func:`paged_attention`."""
     _need(q, "q", torch.bfloat16); _need(k_pages, "k_pages", q.dtype); _need(v_pages, "v_pages", q.dtype)
     for t, nm in ((block_table, "block_table"), (cu_seqlens, "cu_seqlens"), (positions, "positions")):
         _need(t, nm, torch.int32)
@@ -1300,7 +1356,12 @@ def prefill_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
         raise KernelError(f"prefill attention does not take nh={nh} nkv={nkv} head_dim={hd}")
     if cu_seqlens.numel() != n_seqs + 1 or block_table.shape[0] < n_seqs:
         raise KernelError("cu_seqlens / block_table do not match the number of requests")
-    if out is None:
+    part_acc = part_ml = None
+    if parts:
+        out = None
+        part_acc = torch.empty((n, nh, 1, hd), dtype=torch.float32, device=q.device)
+        part_ml = torch.empty((n, nh, 1, 2), dtype=torch.float32, device=q.device)
+    elif out is None:
         out = torch.empty_like(q)
     for t, nm in ((slopes, "slopes"), (sink_values, "sink_values")):
         if t is not None:
@@ -1309,11 +1370,11 @@ def prefill_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Ten
                 raise KernelError(f"{nm} needs one number per query head")
     _check(lib().hb_attention_prefill_reshaped(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
                                                block_table.shape[1], _ptr(cu_seqlens), _ptr(positions), _ptr(out), n_seqs,
-                                               int(max_new), nh, nkv, hd, page_size, int(chunk), int(window), float(scale),
+                                               int(max_new), nh, nkv, hd, page_size, int(chunk), int(window), int(keep), float(scale),
                                                int(skip_single), int(bool(sink) or sink_values is not None),
-                                               float(softcap), _ptr(slopes), _ptr(sink_values), _stream()),
+                                               float(softcap), _ptr(slopes), _ptr(sink_values), _ptr(part_acc), _ptr(part_ml), _stream()),
            "attention_prefill")
-    return out
+    return (part_acc, part_ml) if parts else out
 
 
 PREFILL_TC_MIN_TOKENS = 128     # a request needs at least a tile of new tokens for the tcgen05 kernel to pay
@@ -1331,10 +1392,10 @@ def prefill_attention_tc(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
                          window: int, scale: float, skip_single: bool = False,
                          out: Optional[torch.Tensor] = None, key_splits: int = 1, sink: bool = False,
                          softcap: float = 0.0, slopes: Optional[torch.Tensor] = None,
-                         sink_values: Optional[torch.Tensor] = None) -> torch.Tensor:
+                         sink_values: Optional[torch.Tensor] = None, keep: int = 0) -> torch.Tensor:
     """As :func:`prefill_attention`, on tcgen05 (S, P V and O in tensor memory, TMA page loads).
     ``key_splits`` > 1: that many blocks share the key tiles of every (query tile, head) and a
-    merge kernel combines their rows (see :func:`prefill_key_splits`). ``softcap``, ``slopes``, ``sink_values``:
+    merge kernel combines their rows (see :func:`prefill_key_splits`). ``softcap``, ``slopes``, ``sink_values``, ``keep``:
     as :func:`paged_attention`."""
     _need(q, "q", torch.bfloat16); _need(k_pages, "k_pages", q.dtype); _need(v_pages, "v_pages", q.dtype)
     for t, nm in ((block_table, "block_table"), (cu_seqlens, "cu_seqlens"), (positions, "positions")):
@@ -1360,11 +1421,11 @@ def prefill_attention_tc(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
             if t.numel() != nh:
                 raise KernelError(f"{nm} needs one number per query head")
     sink = bool(sink) or sink_values is not None
-    if softcap or slopes is not None or sink_values is not None:
+    if softcap or slopes is not None or sink_values is not None or keep > 0:
         _check(lib().hb_attention_prefill_tc_reshaped(
             _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], _ptr(cu_seqlens),
             _ptr(positions), _ptr(out), n, n_pages, n_seqs, int(max_new), nh, nkv, hd, page_size, int(chunk), int(window),
-            float(scale), int(skip_single), int(sink), float(softcap), _ptr(slopes), _ptr(sink_values), key_splits,
+            int(keep), float(scale), int(skip_single), int(sink), float(softcap), _ptr(slopes), _ptr(sink_values), key_splits,
             _ptr(part_acc), _ptr(part_ml), _ptr(_tc_status(q.device)), _stream()), "attention_prefill_tc")
     else:
         _check(lib().hb_attention_prefill_tc(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
@@ -1380,6 +1441,173 @@ def prefill_attention_tc(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
         _check(lib().hb_attention_merge(_ptr(part_acc), _ptr(part_ml), _ptr(out), _dt(out), n * nh, hd, key_splits,
                                         int(sink), nh, _ptr(sink_values), _stream()), "attention_merge")
     return out
+
+
+def _gate_args(gate: Optional[torch.Tensor], width: int, dtype: torch.dtype):
+    if gate is None:
+        return None, 0
+    if not gate.is_cuda or gate.dtype != dtype or gate.dim() != 2 or gate.shape[1] != width or gate.stride(1) != 1:
+        raise KernelError(f"the gate must be {dtype} rows of {width} on the device")
+    return _ptr(gate), gate.stride(0)
+
+
+def diff_prefill_attention_tc(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
+                              cu_seqlens: torch.Tensor, positions: torch.Tensor, n_seqs: int, max_new: int, chunk: int,
+                              window: int, keep: int, scale: float, lam: float, eps: float, mul: float, vdim: int,
+                              gate: Optional[torch.Tensor], skip_single: bool = False) -> torch.Tensor:
+    """Differential attention for portions of prompts on tcgen05: heads 2a and 2a + 1 of ``q`` [N, 2H, hd] are the two
+    maps of head a over the same key and value rows; a block takes both, and its epilogue gives
+    o = a1 - lam a2, o <- o rsqrt(mean(o^2) + eps) mul over the head's ``vdim`` values, times sigmoid(``gate``)
+    ([N, H * vdim] rows or None). Returns bfloat16 [N, H * vdim]; with ``skip_single`` the rows of requests that bring
+    one token are unwritten."""
+    _need(q, "q", torch.bfloat16); _need(k_pages, "k_pages", q.dtype); _need(v_pages, "v_pages", q.dtype)
+    for t, nm in ((block_table, "block_table"), (cu_seqlens, "cu_seqlens"), (positions, "positions")):
+        _need(t, nm, torch.int32)
+    n, nh, hd = q.shape
+    n_pages, nkv, page_size, hd2 = k_pages.shape
+    if hd2 != hd or k_pages.shape != v_pages.shape or nh % 2:
+        raise KernelError("cache pages do not match the query's pairs of heads")
+    if not prefill_attention_tc_supported(q.dtype, nh, nkv, hd, page_size):
+        raise KernelError(f"tcgen05 prefill attention does not take nh={nh} nkv={nkv} head_dim={hd} page={page_size}")
+    if cu_seqlens.numel() != n_seqs + 1 or block_table.shape[0] < n_seqs:
+        raise KernelError("cu_seqlens / block_table do not match the number of requests")
+    out = torch.empty((n, nh // 2 * vdim), dtype=q.dtype, device=q.device)
+    g, g_stride = _gate_args(gate, nh // 2 * vdim, q.dtype)
+    _check(lib().hb_diff_prefill_tc(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
+                                    _ptr(cu_seqlens), _ptr(positions), _ptr(out), n, n_pages, n_seqs, int(max_new), nh, nkv,
+                                    hd, page_size, int(chunk), int(window), int(keep), float(scale), int(skip_single),
+                                    float(lam), float(eps), float(mul), int(vdim), g, g_stride, _ptr(_tc_status(q.device)),
+                                    _stream()), "diff_prefill_tc")
+    TC_USED[0] = True
+    return out
+
+
+def diff_merge(part_acc: torch.Tensor, part_ml: torch.Tensor, lam: float, eps: float, mul: float, vdim: int,
+               gate: Optional[torch.Tensor], out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The last step of differential attention from the split partials of its maps (``parts`` of the attention
+    kernels, [R, 2H, splits, hd]): merge, subtract, norm, gate as :func:`diff_prefill_attention_tc` into ``out``
+    [N, H * vdim]. ``rows`` (int64 [R]): row r of the partials belongs to row rows[r] of ``out`` and of the gate."""
+    _need(part_acc, "part_acc", torch.float32); _need(part_ml, "part_ml", torch.float32); _need(out, "out")
+    r, nh, splits, hd = part_acc.shape
+    if nh % 2 or tuple(part_ml.shape) != (r, nh, splits, 2) or out.shape[1] != nh // 2 * vdim:
+        raise KernelError("the partials do not match out")
+    if rows is not None:
+        _need(rows, "rows", torch.int64)
+    if (r if rows is None else rows.numel()) != r or (rows is None and out.shape[0] < r):
+        raise KernelError("one row of out per row of the partials")
+    g, g_stride = _gate_args(gate, nh // 2 * vdim, out.dtype)
+    _check(lib().hb_diff_merge(_ptr(part_acc), _ptr(part_ml), _ptr(rows), g, g_stride, _ptr(out), _dt(out), r, nh // 2, hd,
+                               int(vdim), splits, float(lam), float(eps), float(mul), _stream()), "diff_merge")
+    return out
+
+
+def gate_rows(o: torch.Tensor, gate: torch.Tensor, vdim: int) -> torch.Tensor:
+    """o [N, H, hd] -> [N, H * vdim]: the first ``vdim`` values of every head times sigmoid(gate) ([N, H * vdim] rows)."""
+    _need(o, "o")
+    n, heads, hd = o.shape
+    out = torch.empty((n, heads * vdim), dtype=o.dtype, device=o.device)
+    g, g_stride = _gate_args(gate, heads * vdim, o.dtype)
+    _check(lib().hb_gate_rows(_ptr(o), heads * hd, g, g_stride, _ptr(out), _dt(o), n, heads, hd, int(vdim), _stream()), "gate_rows")
+    return out
+
+
+def conv_qkv(proj: torch.Tensor, taps: Optional[torch.Tensor], state: Optional[torch.Tensor], norm: bool, eps: float,
+             q_norm_weight: Optional[torch.Tensor], k_norm_weight: Optional[torch.Tensor],
+             inv_freq: Optional[torch.Tensor], interleaved: bool, rot_mul: float, positions: torch.Tensor,
+             seq_of_token: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor, block_table: torch.Tensor,
+             k_pages: torch.Tensor, v_pages: torch.Tensor, write_kv: bool, single_tokens: bool, heads: int, kv_heads: int,
+             maps: int, dim: int, vdim: int) -> torch.Tensor:
+    """Short causal convolution over time of the projected channels, RMS norm of q and k per vector, rotation, cache
+    append. ``proj`` [N, >= channels] has the unpadded rows [q: heads * maps * dim | k: kv_heads * maps * dim |
+    v: kv_heads * vdim | ...]; ``taps`` float32 [channels, K] or None; ``state`` float32 [slots, (K - 1) * channels] is
+    read and moved on. Returns q [N, heads * maps, hd] with hd the pages' row length: a map's query at its place of the
+    row, zeros elsewhere; key rows are [map 1 | map 2 | zeros], value rows [vdim | zeros]."""
+    if not proj.is_cuda or proj.dim() != 2 or proj.stride(1) != 1:
+        raise KernelError("proj must be rows on the device")
+    for t, nm in ((positions, "positions"), (seq_of_token, "seq_of_token"), (cu_seqlens, "cu_seqlens"), (slots, "slots"),
+                  (block_table, "block_table")):
+        _need(t, nm, torch.int32)
+    _need(k_pages, "k_pages", proj.dtype); _need(v_pages, "v_pages", proj.dtype)
+    n = proj.shape[0]
+    _, nkv, page_size, hd = k_pages.shape
+    channels = (heads + kv_heads) * maps * dim + kv_heads * vdim
+    if nkv != kv_heads or k_pages.shape != v_pages.shape or max(maps * dim, vdim) > hd or proj.shape[1] < channels:
+        raise KernelError("proj or the cache pages do not match the heads")
+    taps_n, state_stride = 1, 0
+    if taps is not None:
+        _need(taps, "taps", torch.float32)
+        taps_n = taps.shape[1]
+        if taps.shape[0] != channels:
+            raise KernelError(f"taps for {taps.shape[0]} channels, the projection has {channels}")
+        if taps_n > 1:
+            _need(state, "state", torch.float32)
+            state_stride = state.shape[1]
+            if state_stride < (taps_n - 1) * channels:
+                raise KernelError("the state rows are too short for the convolution's inputs")
+    for t, nm in ((q_norm_weight, "q_norm_weight"), (k_norm_weight, "k_norm_weight")):
+        if t is not None:
+            _need(t, nm, torch.float32)
+            if t.numel() != dim:
+                raise KernelError(f"{nm} needs one weight per dim of a head ({dim})")
+    if inv_freq is not None:
+        _need(inv_freq, "inv_freq", torch.float32)
+    q = torch.empty((n, heads * maps, hd), dtype=proj.dtype, device=proj.device)
+    moved = c_int(0)
+    _check(lib().hb_conv_qkv(_ptr(proj), _dt(proj), proj.stride(0), _ptr(taps), taps_n, _ptr(state) if taps_n > 1 else None,
+                             state_stride, 0, int(norm), float(eps), _ptr(q_norm_weight), _ptr(k_norm_weight),
+                             _ptr(inv_freq), 0 if inv_freq is None else inv_freq.numel(), int(interleaved), float(rot_mul),
+                             _ptr(positions), _ptr(seq_of_token), _ptr(cu_seqlens), _ptr(slots), _ptr(block_table),
+                             block_table.shape[1], _ptr(q), _ptr(k_pages), _ptr(v_pages), page_size, int(write_kv),
+                             int(single_tokens), n, heads, kv_heads, maps, dim, vdim, hd, ctypes.byref(moved), _stream()),
+           "conv_qkv")
+    if taps_n > 1 and not moved.value and n:
+        delta_conv_update(proj, 0, channels, taps_n, state, 0, cu_seqlens, slots)
+    return q
+
+
+def sandwich_step(x: torch.Tensor, y_weight: torch.Tensor, y_eps: float, delta: Optional[torch.Tensor] = None,
+                  delta2: Optional[torch.Tensor] = None, routed: Optional[torch.Tensor] = None,
+                  slot_of_entry: Optional[torch.Tensor] = None, top_k: int = 0,
+                  routed_weight: Optional[torch.Tensor] = None, weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+                  out_dtype: Optional[torch.dtype] = None, row_map: Optional[torch.Tensor] = None, also_f32: bool = False):
+    """``x += rmsnorm(delta + delta2 + routed rows) * y_weight`` (float32, in place), then, with ``weight``,
+    ``rmsnorm(x) * weight`` in ``out_dtype`` (returned; None without ``weight``). ``routed``, ``slot_of_entry``,
+    ``routed_weight``, ``row_map`` and ``also_f32`` as :func:`add_rmsnorm`; the weights are float32."""
+    _need(x, "x", torch.float32); _need(y_weight, "y_weight", torch.float32)
+    rows_total, hidden = x.shape
+    for t, nm in ((delta, "delta"), (delta2, "delta2")):
+        if t is not None:
+            _need(t, nm)
+            if t.shape != x.shape:
+                raise KernelError(f"{nm} shape {tuple(t.shape)} != residual shape {tuple(x.shape)}")
+    for t, nm in ((y_weight, "y_weight"), (weight, "weight")):
+        if t is not None:
+            _need(t, nm, torch.float32)
+            if t.numel() != hidden:
+                raise KernelError(f"{nm} has {t.numel()} elements for hidden size {hidden}")
+    rows = rows_total
+    if row_map is not None:
+        _need(row_map, "row_map", torch.int32)
+        rows = row_map.numel()
+    if routed is not None:
+        _need(routed, "routed", torch.float32); _need(slot_of_entry, "slot_of_entry", torch.int32)
+        if routed.shape[1] != hidden or not 1 <= top_k <= 8:
+            raise KernelError("routed rows do not match the residual, or top_k is outside 1..8")
+        if routed_weight is not None:
+            _need(routed_weight, "routed_weight", torch.float32)
+    y = y32 = None
+    if weight is not None:
+        y = torch.empty((rows, hidden), dtype=out_dtype, device=x.device)
+        if also_f32 and out_dtype != torch.float32:
+            y32 = torch.empty((rows, hidden), dtype=torch.float32, device=x.device)
+    _check(lib().hb_sandwich_step(_ptr(x), _ptr(delta), _dt(delta) if delta is not None else 0, _ptr(delta2),
+                                  _dt(delta2) if delta2 is not None else 0, _ptr(routed), _ptr(slot_of_entry),
+                                  _ptr(routed_weight) if routed is not None else None, int(top_k), _ptr(y_weight),
+                                  float(y_eps), _ptr(weight), float(eps), _ptr(y), _dt(y) if y is not None else 0, _ptr(y32),
+                                  _ptr(row_map), rows, hidden, _stream()), "sandwich_step")
+    if also_f32:
+        return y, (y if y32 is None else y32)
+    return y
 
 
 _sm_counts: dict = {}
@@ -1431,10 +1659,11 @@ def router_groups(count: int, keep: int) -> int:
 
 
 def router_topk(x: torch.Tensor, w: torch.Tensor, top_k: int, want_logits: bool = False, mode: int = 0,
-                score_scale: float = 1.0):
+                score_scale: float = 1.0, bias: Optional[torch.Tensor] = None):
     """Router logits (float32), the top-k expert ids (ties to the lower id) and their scores: the
     sigmoid of the chosen logit, or with ``ROUTER_SOFTMAX`` its softmax over all experts; with
-    ``ROUTER_RENORMALIZE`` divided by the sum of the chosen scores."""
+    ``ROUTER_RENORMALIZE`` divided by the sum of the chosen scores (together: the softmax over the chosen logits).
+    ``bias`` (float32 [experts]) is added to the logits first."""
     _need(x, "x"); _need(w, "router weight")
     n, hidden = x.shape
     experts = w.shape[0]
@@ -1443,7 +1672,7 @@ def router_topk(x: torch.Tensor, w: torch.Tensor, top_k: int, want_logits: bool 
     ids = torch.empty((n, top_k), dtype=torch.int32, device=x.device)
     scores = torch.empty((n, top_k), dtype=torch.float32, device=x.device)
     logits = torch.empty((n, experts), dtype=torch.float32, device=x.device)   # the blocks' meeting place
-    _check(lib().hb_router_topk(_ptr(x), _dt(x), _ptr(w), _dt(w), n, hidden, experts, top_k, int(mode), float(score_scale),
+    _check(lib().hb_router_topk(_ptr(x), _dt(x), _ptr(w), _dt(w), _router_bias(bias, experts), n, hidden, experts, top_k, int(mode), float(score_scale),
                                 _ptr(logits), _ptr(ids), _ptr(scores), _stream()), "router_topk")
     return ids, scores, logits if want_logits else None
 
@@ -1479,7 +1708,16 @@ def _block_counter(dev) -> torch.Tensor:
     return c
 
 
-def router_plan(x: torch.Tensor, w: torch.Tensor, top_k: int, mode: int = 0, score_scale: float = 1.0):
+def _router_bias(bias: Optional[torch.Tensor], experts: int):
+    if bias is not None:
+        _need(bias, "router bias", torch.float32)
+        if bias.numel() != experts:
+            raise KernelError("one router bias per expert")
+    return _ptr(bias)
+
+
+def router_plan(x: torch.Tensor, w: torch.Tensor, top_k: int, mode: int = 0, score_scale: float = 1.0,
+                bias: Optional[torch.Tensor] = None):
     """:func:`router_topk` and :func:`moe_plan` in one call: with few tokens one kernel does both
     (the block that ends last groups the entries). Returns ids, scores and the plan."""
     _need(x, "x"); _need(w, "router weight")
@@ -1491,7 +1729,7 @@ def router_plan(x: torch.Tensor, w: torch.Tensor, top_k: int, mode: int = 0, sco
     scores = torch.empty((n, top_k), dtype=torch.float32, device=x.device)
     logits = torch.empty((n, experts), dtype=torch.float32, device=x.device)   # the blocks' meeting place
     plan = _empty_plan(n * top_k, experts, x.device)
-    _check(lib().hb_router_plan(_ptr(x), _dt(x), _ptr(w), _dt(w), n, hidden, experts, top_k, int(mode), float(score_scale),
+    _check(lib().hb_router_plan(_ptr(x), _dt(x), _ptr(w), _dt(w), _router_bias(bias, experts), n, hidden, experts, top_k, int(mode), float(score_scale),
                                 _ptr(logits), _ptr(ids), _ptr(scores), _ptr(plan.offsets), _ptr(plan.sorted_entry),
                                 _ptr(plan.slot_of_entry), _ptr(plan.active), _ptr(_block_counter(x.device)),
                                 _stream()), "router_plan")
@@ -1508,13 +1746,18 @@ def moe_plan(ids: torch.Tensor, experts: int) -> MoePlan:
     return plan
 
 
+EXPERT_ACTIVATIONS = ("swiglu", "relu2", "clamped")
+
+
 def moe_gate_up(x: torch.Tensor, plan: MoePlan, top_k: int, w_gate: Optional[torch.Tensor],
-                w_up: torch.Tensor, scores: torch.Tensor, few_rows: bool, activation: str = "swiglu") -> torch.Tensor:
+                w_up: torch.Tensor, scores: torch.Tensor, few_rows: bool, activation: str = "swiglu",
+                limit: float = 0.0) -> torch.Tensor:
     """act[slot] = silu(s * x Wg[e]^T) * (s * x Wu[e]^T), [N*k, I] in the engine dtype; with
-    ``activation="relu2"`` (experts without a gate branch; ``w_gate`` None) max(s * x Wu[e]^T, 0)^2."""
+    ``activation="relu2"`` (experts without a gate branch; ``w_gate`` None) max(s * x Wu[e]^T, 0)^2; with
+    ``activation="clamped"`` min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, +-limit) + 1)."""
     _need(x, "x"); _need(w_up, "w_up", x.dtype)
     _need(scores, "scores", torch.float32)
-    if activation not in ("swiglu", "relu2") or (w_gate is None) != (activation == "relu2"):
+    if activation not in EXPERT_ACTIVATIONS or (w_gate is None) != (activation == "relu2"):
         raise KernelError("experts have a gate stack with swiglu and none with relu2")
     n, hidden = x.shape
     experts, inter, h2 = w_up.shape
@@ -1526,7 +1769,7 @@ def moe_gate_up(x: torch.Tensor, plan: MoePlan, top_k: int, w_gate: Optional[tor
     act = torch.empty((n_entries, inter), dtype=x.dtype, device=x.device)
     _check(lib().hb_moe_gate_up(_ptr(x), _dt(x), _ptr(plan.sorted_entry), top_k, _ptr(w_gate), _ptr(w_up),
                                 _ptr(plan.offsets), _ptr(plan.active), experts, _ptr(scores), _ptr(act), n_entries,
-                                inter, hidden, int(few_rows), 1 if activation == "relu2" else 0, _stream()),
+                                inter, hidden, int(few_rows), EXPERT_ACTIVATIONS.index(activation), float(limit), _stream()),
            "moe_gate_up")
     return act
 
@@ -1628,9 +1871,9 @@ def gather_rows(x: torch.Tensor, plan: MoePlan, top_k: int) -> torch.Tensor:
 
 
 def moe_gate_up_tc(x: torch.Tensor, plan: MoePlan, top_k: int, w_gate: torch.Tensor, w_up: torch.Tensor,
-                   scores: torch.Tensor) -> torch.Tensor:
+                   scores: torch.Tensor, limit: float = 0.0) -> torch.Tensor:
     """As :func:`moe_gate_up`, on tcgen05: gathers the rows into expert order, then one grouped
-    product with the SwiGLU epilogue."""
+    product with the SwiGLU epilogue (``limit`` > 0: the clamped unit's)."""
     _need(x, "x", torch.bfloat16); _need(w_gate, "w_gate", torch.bfloat16); _need(w_up, "w_up", torch.bfloat16)
     _need(scores, "scores", torch.float32)
     n, hidden = x.shape
@@ -1643,7 +1886,7 @@ def moe_gate_up_tc(x: torch.Tensor, plan: MoePlan, top_k: int, w_gate: torch.Ten
            "gather_rows")
     act = torch.empty((rows, inter), dtype=x.dtype, device=x.device)
     _check(lib().hb_moe_gate_up_tc(_ptr(xs), _ptr(plan.sorted_entry), _ptr(w_gate), _ptr(w_up), _ptr(plan.offsets),
-                                   experts, _ptr(scores), _ptr(act), rows, inter, hidden, _ptr(_tc_status(x.device)),
+                                   experts, _ptr(scores), _ptr(act), rows, inter, hidden, float(limit), _ptr(_tc_status(x.device)),
                                    _stream()), "moe_gate_up_tc")
     TC_USED[0] = True
     return act

@@ -8,7 +8,7 @@ import numpy as np
 import torch
 
 from ..kernels import ops
-from .context import GatedPending, HyperPending, Pending
+from .context import GatedPending, HyperPending, NormedPending, Pending
 from .linear import linear
 from .registry import BuildEnv, build, register
 from .spec import PartSpec, TensorSpec
@@ -59,6 +59,7 @@ class RMSNorm(Part):
         self.size, self.eps = int(params["size"]), float(params["eps"])
         self.one_plus = bool(params.get("one_plus", False))
         self.weight: Optional[torch.Tensor] = None
+        self.weight_f32: Optional[torch.Tensor] = None
         self.tensor_name = prefix if params.get("tensor") == "bare" else f"{prefix}.weight"
 
     def tensor_specs(self):
@@ -67,6 +68,7 @@ class RMSNorm(Part):
     def load(self, fetch):
         w = fetch(self.tensor_name)
         self.weight = (w.to(torch.float32) + 1.0).contiguous() if self.one_plus else w.contiguous()
+        self.weight_f32 = self.weight.to(torch.float32)
 
     def forward(self, residual: torch.Tensor, delta, row_map: Optional[torch.Tensor] = None, also_f32: bool = False,
                 out_dtype: Optional[torch.dtype] = None):
@@ -75,6 +77,10 @@ class RMSNorm(Part):
         out_dtype = out_dtype or self.env.dtype
         if isinstance(delta, HyperPending):
             return resolve_hyper(residual, delta, self.weight, self.eps, out_dtype, None, row_map, also_f32)
+        if isinstance(delta, NormedPending):
+            return ops.sandwich_step(residual, delta.weight, delta.eps, weight=self.weight_f32, eps=self.eps,
+                                     out_dtype=out_dtype, row_map=row_map, also_f32=also_f32,
+                                     **delta.parts(residual.shape[0]))
         if isinstance(delta, Pending):
             if delta.top_k > 8:
                 delta = delta.materialize(residual.shape[0])
@@ -120,6 +126,9 @@ class DynamicTanh(Part):
         """The stream after ``pending`` and the outputs of up to two norms of it, in one kernel:
         ``(stream | None, [y])``. Without a ``GatedPending`` the stream is ``residual`` itself."""
         triples = [n.triple() for n in norms]
+        if isinstance(pending, NormedPending):
+            pending.resolve(residual)
+            pending = None
         if isinstance(pending, GatedPending):
             z, ys = ops.gated_depth_dyt(residual, pending.terms, pending.history, pending.filled, pending.mix,
                                         triples, out_dtype, row_map, want_z=want_stream)
@@ -285,7 +294,9 @@ class NoPosition(Part):
 @register("embedding", "token_embedding")
 class TokenEmbedding(Part):
     """x[t] = table[token[t]] * scale; no multiplier by default (crates/hi-mlx/src/models.rs:6206, 1915-1917).
-    params: ``vocab_size``, ``hidden_size``, ``scale`` (default 1); tensor ``<prefix>.weight``."""
+    params: ``vocab_size``, ``hidden_size``, ``scale`` (default 1), ``sinusoid`` (None, or a base b: a vector of the
+    token's absolute position p is added, entry 2i sin(p b^(-2i/hidden)), entry 2i + 1 the cosine of the same angle;
+    angles are worked out in float64 and reduced to a turn before sine and cosine); tensor ``<prefix>.weight``."""
 
     graph_safe = True
 
@@ -293,14 +304,23 @@ class TokenEmbedding(Part):
         super().__init__(params, prefix, env)
         self.table: Optional[torch.Tensor] = None
         self.scale = float(params.get("scale", 1.0))
+        self.sinusoid = float(params["sinusoid"]) if params.get("sinusoid") else None
+        self.needs_positions = self.sinusoid is not None
+        self._turns: Optional[torch.Tensor] = None
 
     def tensor_specs(self):
         return [TensorSpec(f"{self.prefix}.weight", (int(self.params["vocab_size"]), int(self.params["hidden_size"])))]
 
     def load(self, fetch):
         self.table = fetch(f"{self.prefix}.weight").contiguous()
+        if self.sinusoid is not None:
+            h = int(self.params["hidden_size"])
+            turns = [self.sinusoid ** (-2.0 * i / h) / (2.0 * math.pi) for i in range((h + 1) // 2)]
+            self._turns = torch.tensor(turns, dtype=torch.float64).to(self.table.device)
 
-    def forward(self, tokens: torch.Tensor) -> torch.Tensor:
+    def forward(self, tokens: torch.Tensor, positions: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if self.sinusoid is not None:
+            return ops.embed_position(self.table, tokens, positions, self._turns, scale=self.scale)
         return ops.embed_gather(self.table, tokens, scale=self.scale)
 
 
@@ -415,6 +435,55 @@ class PostNormBlock(Part):
         if ctx.tap is not None:
             ctx.tap(f"{self.prefix}.stream_out", residual)
         return residual, None
+
+
+@register("arrangement", "sandwich")
+class SandwichBlock(Part):
+    """A norm before and one after each sub-layer: x <- x + norm1b(mixer(norm1(x))); x <- x + norm2b(ff(norm2(x))).
+
+    The residual stream is float32. A sub-layer's result stays open until the next norm, which takes it through its
+    own norm, sums it into the stream and norms the sum for the next sub-layer in one kernel
+    (:class:`~hi_b200.parts.context.NormedPending`). A layer without feed-forward has the first half only.
+
+    params: ``hidden_size``, ``eps``, ``one_plus`` (weights stored around zero), ``feed_forward`` (default True).
+    tensors: ``<prefix>.norm1b``, ``<prefix>.norm2b`` [W]. The norms of the layer must be ``rmsnorm``."""
+
+    graph_safe = True
+
+    def __init__(self, params, prefix, env):
+        super().__init__(params, prefix, env)
+        self.has_ff = bool(params.get("feed_forward", True))
+        spec = {"size": int(params["hidden_size"]), "eps": float(params["eps"]), "tensor": "bare",
+                "one_plus": bool(params.get("one_plus", False))}
+        self.after = [RMSNorm(spec, f"{prefix}.{n}", env) for n in (("norm1b", "norm2b") if self.has_ff else ("norm1b",))]
+
+    def tensor_specs(self):
+        return [t for n in self.after for t in n.tensor_specs()]
+
+    def load(self, fetch):
+        for n in self.after:
+            n.load(fetch)
+
+    def _open(self, which: int, delta):
+        norm = self.after[which]
+        return NormedPending(delta=delta, weight=norm.weight_f32, eps=norm.eps)
+
+    def forward(self, layer, residual, pending, ctx, cache_view):
+        if not isinstance(layer.norm_mixer, RMSNorm) or (self.has_ff and not isinstance(layer.norm_feed_forward, RMSNorm)):
+            raise TypeError(f"{self.prefix}: the block works with rmsnorm norms")
+        h = layer.norm_mixer.forward(residual, pending)
+        if ctx.tap is not None:
+            ctx.tap(f"{self.prefix}.stream_in", residual)        # debug: the stream as this layer reads it
+        pending = self._open(0, layer.mixer.forward(h, ctx, cache_view))
+        if self.has_ff:
+            if getattr(layer.feed_forward, "wants_f32_input", False):
+                h, h32 = layer.norm_feed_forward.forward(residual, pending, also_f32=True)
+                y = layer.feed_forward.forward(h, ctx, normed_f32=h32)
+            else:
+                h = layer.norm_feed_forward.forward(residual, pending)
+                y = layer.feed_forward.forward(h, ctx)
+            pending = self._open(1, y)
+        return residual, pending
 
 
 _side_streams: Dict[torch.device, "torch.cuda.Stream"] = {}
@@ -722,6 +791,9 @@ class PassOffset(Part):
 
     def forward(self, residual, pending, ctx, arg: int):
         d1 = d2 = None
+        if isinstance(pending, NormedPending):
+            pending.resolve(residual)
+            pending = None
         if isinstance(pending, Pending):
             if pending.routed is not None:
                 d1 = pending.materialize(residual.shape[0])

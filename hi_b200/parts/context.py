@@ -104,6 +104,33 @@ class GatedPending:
 
 
 @dataclass
+class NormedPending:
+    """What a block that norms its sub-layers' results leaves for the next norm: a result (``delta``: a tensor or a
+    :class:`Pending`) that enters the stream as rmsnorm(delta) * weight (``weight`` float32). The norm that takes it
+    does both in one kernel (``ops.sandwich_step``)."""
+
+    delta: object
+    weight: torch.Tensor
+    eps: float
+
+    def parts(self, n_tokens: int) -> dict:
+        """The open result as the kernel's arguments."""
+        d = self.delta
+        if isinstance(d, Pending) and d.top_k > 8:
+            d = d.materialize(n_tokens)
+        if not isinstance(d, Pending):
+            return {"delta": d}
+        return {"delta": d.dense, "delta2": d.dense2, "routed": d.routed, "slot_of_entry": d.slot_of_entry,
+                "top_k": d.top_k, "routed_weight": d.entry_weights}
+
+    def resolve(self, residual: torch.Tensor) -> None:
+        """Into the stream, for a consumer that is not an RMS norm."""
+        from ..kernels import ops
+
+        ops.sandwich_step(residual, self.weight, self.eps, **self.parts(residual.shape[0]))
+
+
+@dataclass
 class HyperPending:
     """What a block with a residual stream of several copies leaves for the next norm: a sub-layer's result
     (``delta``: a tensor or a :class:`Pending`) and the coefficients it enters the copies with,

@@ -15,9 +15,18 @@ from .spec import TensorSpec
 
 class _SwiGLU:
     """(silu(x Wg^T) * x Wu^T) Wd^T with gate and up fused into one product
-    (Mlp::forward, crates/hi-mlx/src/models.rs:2307-2312)."""
+    (Mlp::forward, crates/hi-mlx/src/models.rs:2307-2312).
 
-    def __init__(self, prefix: str, hidden: int, inter: int, short_names: bool = False):
+    ``limit``: the clamped unit instead, min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, +-limit) + 1).
+    ``token_gate``: the result of every token is multiplied by sigmoid(Ws x), one number a token (tensor
+    ``<prefix>.sg`` [1, H]); Ws rides in the product as one more row, and the factor goes on the activation, in front
+    of the down projection."""
+
+    def __init__(self, prefix: str, hidden: int, inter: int, short_names: bool = False, limit: Optional[float] = None,
+                 token_gate: bool = False):
+        self.limit, self.token_gate = limit, token_gate
+        if token_gate and limit is None:
+            raise ValueError(f"{prefix}: a gate per token is built for the clamped unit")
         self.prefix, self.hidden, self.inter = prefix, hidden, inter
         self.suffix = "" if short_names else "_proj.weight"
         self.w_gate_up: Optional[torch.Tensor] = None
@@ -29,16 +38,23 @@ class _SwiGLU:
     def tensor_specs(self):
         return [TensorSpec(self._name("gate"), (self.inter, self.hidden)),
                 TensorSpec(self._name("up"), (self.inter, self.hidden)),
-                TensorSpec(self._name("down"), (self.hidden, self.inter))]
+                TensorSpec(self._name("down"), (self.hidden, self.inter))] + \
+            ([TensorSpec(f"{self.prefix}.sg", (1, self.hidden))] if self.token_gate else [])
 
     def load(self, fetch):
-        g, u = fetch(self._name("gate")), fetch(self._name("up"))
-        if g.dtype != u.dtype:
-            g, u = g.float(), u.float()
-        self.w_gate_up = torch.cat([g, u], dim=0).contiguous()
+        rows = [fetch(self._name("gate")), fetch(self._name("up"))]
+        if self.token_gate:      # one more row, and zero rows up to a multiple of eight (rows of the product stay 16-byte aligned)
+            sg = fetch(f"{self.prefix}.sg")
+            rows += [sg, torch.zeros((-(2 * self.inter + 1) % 8, self.hidden), dtype=sg.dtype, device=sg.device)]
+        if len({t.dtype for t in rows}) > 1:
+            rows = [t.float() for t in rows]
+        self.w_gate_up = torch.cat(rows, dim=0).contiguous()
         self.w_down = fetch(self._name("down")).contiguous()
 
     def forward(self, x):
+        if self.limit is not None:
+            return linear(ops.glu_limit(linear(x, self.w_gate_up), self.inter, self.limit,
+                                        2 * self.inter if self.token_gate else -1), self.w_down)
         return linear(ops.swiglu(linear(x, self.w_gate_up)), self.w_down)
 
 
@@ -73,10 +89,11 @@ class DenseMLP(Part):
       "xielu"  z > 0: softplus(p) z^2 + z/2;  z <= 0: (1/2 + softplus(q)) (e^z - 1 - z) + z/2, with the
                two learned numbers (p, q) of ``<prefix>.act``; the coefficients are worked out once, in float32.
       "relu2"  max(z, 0)^2; no tensor of its own
+      "gelu"   0.5 z (1 + erf(z / sqrt 2)); no tensor of its own
     tensors: ``<prefix>.up`` [I, H], ``<prefix>.down`` [H, I], ``<prefix>.act`` [2] (xielu)."""
 
     graph_safe = True
-    ACTIVATIONS = ("xielu", "relu2")
+    ACTIVATIONS = ("xielu", "relu2", "gelu")
 
     def __init__(self, params, prefix, env):
         super().__init__(params, prefix, env)
@@ -102,7 +119,9 @@ class DenseMLP(Part):
 
     def forward(self, normed, ctx):
         z = linear(normed, self.w_up)
-        return linear(ops.relu2(z) if self.activation == "relu2" else ops.xielu(z, self.coef), self.w_down)
+        if self.activation == "xielu":
+            return linear(ops.xielu(z, self.coef), self.w_down)
+        return linear(ops.relu2(z) if self.activation == "relu2" else ops.gelu(z), self.w_down)
 
 
 @register("feed_forward", "routed_experts")
@@ -121,7 +140,12 @@ class SigmoidRoutedExperts(Part):
       ``scale``        "input" (default: the score multiplies what the expert reads) | "output"
                        (it multiplies what the expert returns, in the sum the next norm takes)
       ``activation``   "swiglu" (default: gate and up stacks) | "relu2" (W_down max(W_up x, 0)^2: no gate stack;
-                       the score then has to scale the output)
+                       the score then has to scale the output) | "clamped" (gate and up stacks with limits:
+                       g = min(gate, ``limit``), u = clamp(up, +-``limit``), g sigmoid(1.702 g) (u + 1))
+      ``router_bias``  a number per expert is added to the router's logits: ``<prefix>.router.b`` [E] (default False)
+      ``shared_limit`` the shared expert is the clamped unit with this limit (default None: SwiGLU)
+      ``shared_gate``  the shared expert's result is multiplied by sigmoid(W x), one number a token:
+                       ``<prefix>.shared.sg`` [1, H] (default False)
       ``groups``       None | (count, keep): the experts lie in ``count`` equal groups of neighbours, a group
                        counts as the sum of its two largest scores, and only experts of the ``keep`` best
                        groups can be chosen
@@ -150,8 +174,10 @@ class SigmoidRoutedExperts(Part):
         self.shared = None
         if params.get("shared_expert", True):
             shared_inter = int(params.get("shared_intermediate_size") or self.inter)
-            self.shared = _SwiGLU(f"{prefix}.shared", self.hidden, shared_inter, short_names=True) \
-                if self.per_expert_names else _SwiGLU(f"{prefix}.shared_expert", self.hidden, shared_inter)
+            limit = float(params["shared_limit"]) if params.get("shared_limit") is not None else None
+            self.shared = _SwiGLU(f"{prefix}.shared" if self.per_expert_names else f"{prefix}.shared_expert", self.hidden,
+                                  shared_inter, short_names=self.per_expert_names, limit=limit,
+                                  token_gate=bool(params.get("shared_gate", False)))
         score, scale = params.get("score", "sigmoid"), params.get("scale", "input")
         if score not in ("sigmoid", "softmax") or scale not in ("input", "output"):
             raise ValueError(f"{prefix}: score {score!r} / scale {scale!r} are not known (sigmoid | softmax; input | output)")
@@ -159,9 +185,14 @@ class SigmoidRoutedExperts(Part):
             (ops.ROUTER_RENORMALIZE if params.get("renormalize", False) else 0)
         self.scale_output = scale == "output"
         self.activation = params.get("activation", "swiglu")
-        if self.activation not in ("swiglu", "relu2") or (self.activation == "relu2" and not self.scale_output):
-            raise ValueError(f"{prefix}: activation {self.activation!r} is not known (swiglu | relu2), or relu2 "
-                             f"without scale 'output' (a score on the input would be squared)")
+        if self.activation not in ops.EXPERT_ACTIVATIONS or (self.activation != "swiglu" and not self.scale_output):
+            raise ValueError(f"{prefix}: activation {self.activation!r} is not known {ops.EXPERT_ACTIVATIONS}, or it is not "
+                             f"swiglu and scale is not 'output' (a score on the input would go through the activation)")
+        self.limit = float(params["limit"]) if self.activation == "clamped" else 0.0
+        if self.activation == "clamped" and not self.limit > 0:
+            raise ValueError(f"{prefix}: the clamped unit needs a positive limit")
+        self.router_bias = bool(params.get("router_bias", False))
+        self.b_router: Optional[torch.Tensor] = None
         self.groups = tuple(int(g) for g in params["groups"]) if params.get("groups") else None
         if self.groups:
             count, keep = self.groups
@@ -176,7 +207,7 @@ class SigmoidRoutedExperts(Part):
 
     def tensor_specs(self):
         e, i, h, p = self.experts, self.inter, self.hidden, self.prefix
-        gated = self.activation == "swiglu"
+        gated = self.activation != "relu2"
         if self.per_expert_names:
             specs = [TensorSpec(f"{p}.router", (e, h))]
             for j in range(e):
@@ -187,6 +218,8 @@ class SigmoidRoutedExperts(Part):
                 ([TensorSpec(f"{p}.experts.gate_proj.weight", (e, i, h))] if gated else []) + \
                 [TensorSpec(f"{p}.experts.up_proj.weight", (e, i, h)),
                  TensorSpec(f"{p}.experts.down_proj.weight", (e, h, i))]
+        if self.router_bias:
+            specs.append(TensorSpec(f"{p}.router.b", (e,)))
         return specs + (self.shared.tensor_specs() if self.shared else [])
 
     def load(self, fetch):
@@ -200,7 +233,9 @@ class SigmoidRoutedExperts(Part):
                     f"{self.env.dtype} path cannot take it (run with --dtype float32)")
             return t.contiguous()
 
-        gated = self.activation == "swiglu"
+        gated = self.activation != "relu2"
+        if self.router_bias:
+            self.b_router = fetch(f"{p}.router.b").to(torch.float32).contiguous()
         if self.per_expert_names:
             stack = lambda part: torch.stack([expert_tensor(f"{p}.e{j}.{part}") for j in range(self.experts)]).contiguous()
             self.w_router = expert_tensor(f"{p}.router")
@@ -237,11 +272,12 @@ class SigmoidRoutedExperts(Part):
         router_in = normed if normed_f32 is None else normed_f32
         forced = ctx.forced.get(f"{self.prefix}.router_ids") if ctx.forced else None
         if forced is None:
-            ids, scores, plan = ops.router_plan(router_in, self.w_router, self.top_k, self.router_mode, self.score_scale)
+            ids, scores, plan = ops.router_plan(router_in, self.w_router, self.top_k, self.router_mode, self.score_scale,
+                                                bias=self.b_router)
         else:
             # debug: another run's expert choices, scored with this run's own logits (two runs in
             # different precisions can then be compared token by token)
-            _own, _s, logits = ops.router_topk(router_in, self.w_router, self.top_k, want_logits=True)
+            _own, _s, logits = ops.router_topk(router_in, self.w_router, self.top_k, want_logits=True, bias=self.b_router)
             ids = forced.to(device=logits.device, dtype=torch.int32).reshape(n, self.top_k).contiguous()
             chosen = torch.gather(logits, 1, ids.long())
             scores = torch.sigmoid(chosen) if not self.router_mode & ops.ROUTER_SOFTMAX else \
@@ -265,10 +301,10 @@ class SigmoidRoutedExperts(Part):
             y = ops.moe_down_tc(ops.moe_up_relu2_tc(normed, plan, self.top_k, self.w_up), self.w_down, plan)
         elif not few and tc:
             # many rows per expert: the grouped products run on tcgen05
-            act = ops.moe_gate_up_tc(normed, plan, self.top_k, self.w_gate, self.w_up, scores)
+            act = ops.moe_gate_up_tc(normed, plan, self.top_k, self.w_gate, self.w_up, scores, self.limit)
             y = ops.moe_down_tc(act, self.w_down, plan)
         else:
-            act = ops.moe_gate_up(normed, plan, self.top_k, self.w_gate, self.w_up, scores, few, self.activation)
+            act = ops.moe_gate_up(normed, plan, self.top_k, self.w_gate, self.w_up, scores, few, self.activation, self.limit)
             y = ops.moe_down(act, self.w_down, plan, few)
         if side is not None:
             torch.cuda.current_stream().wait_stream(side)

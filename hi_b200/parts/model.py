@@ -108,7 +108,8 @@ class Model:
         if not self.loaded:
             raise RuntimeError("model weights are not loaded")
         ctx.scratch = {}
-        residual = self.embedding.forward(ctx.tokens)
+        residual = self.embedding.forward(ctx.tokens, ctx.positions) if getattr(self.embedding, "needs_positions", False) \
+            else self.embedding.forward(ctx.tokens)
         if any(getattr(p, "needs_embedding_output", False) for p in self.interludes):
             ctx.scratch["embedding_output"] = residual.clone()       # the stream is summed into in place
         pending = None

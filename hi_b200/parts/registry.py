@@ -12,7 +12,8 @@ Families and the interface each member must have (all also have
                   ``forward(normed, ctx, cache_view) -> delta``.
 ``feed_forward``  ``forward(normed, ctx) -> delta`` (engine dtype or float32).
 ``arrangement``   ``forward(layer, residual, pending, ctx, cache_view) -> (residual, pending)``.
-``embedding``     ``forward(tokens_i32) -> residual_f32``; ``table`` for a tied head.
+``embedding``     ``forward(tokens_i32) -> residual_f32`` (with ``needs_positions``: ``forward(tokens_i32, positions_i32)``);
+                  ``table`` for a tied head.
 ``head``          ``forward(normed_rows) -> logits_f32``.
 ``interlude``     ``forward(residual, pending, ctx, arg) -> (residual, pending)``: acts on the stream between
                   two runs of layers; ``needs_embedding_output`` asks the model to keep a copy of the

@@ -40,7 +40,8 @@ class CacheSpec:
 
     Per token: one key row and one value row of ``kv_heads * head_dim`` elements,
     kept for ``window``: ``None`` = all earlier tokens, ``("chunk", C)`` = tokens of
-    the query's own block of C positions, ``("sliding", W)`` = the last W tokens.
+    the query's own block of C positions, ``("sliding", W)`` = the last W tokens,
+    ``("sliding", W, K)`` = the last W tokens and the first K of the request.
     ``values=False``: the mixer keeps one row per token only (a latent from which it makes
     keys and values itself); no value pool is allocated and its view has ``v_pages`` None.
     Per request: ``state_shape`` elements of fixed size (``()`` = none).
@@ -49,7 +50,7 @@ class CacheSpec:
 
     kv_heads: int = 0
     head_dim: int = 0
-    window: Optional[Tuple[str, int]] = None
+    window: Optional[Tuple] = None
     state_shape: Tuple[int, ...] = ()
     state_dtype: str = "float32"
     values: bool = True
@@ -62,11 +63,16 @@ class CacheSpec:
     def group_key(self):
         return (self.kv_heads, self.head_dim, self.window)
 
+    @property
+    def keep_first(self) -> int:
+        """How many tokens at a request's start stay readable although the window has passed them."""
+        return int(self.window[2]) if self.window is not None and len(self.window) > 2 else 0
+
     def first_live_position(self, next_position: int) -> int:
-        """Oldest position a query at ``next_position`` or later can still read."""
+        """Oldest position a query at ``next_position`` or later can still read (kept first tokens aside)."""
         if self.window is None:
             return 0
-        kind, size = self.window
+        kind, size = self.window[:2]
         if kind == "chunk":
             return (next_position // size) * size
         if kind == "sliding":
