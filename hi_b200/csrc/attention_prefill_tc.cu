@@ -443,16 +443,21 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         tc::st32_nowait(tmem + lane_addr + sb * S_COLS, packed);
         tc::wait_st();
       }
-      if (key_base / BKEYS == p_last / BKEYS && (p_last + 1) % BKEYS != 0) {
-        // Value rows of positions past the portion's end hold whatever the page held before
-        // (another request's numbers, possibly not finite): P is zero there, but 0 x NaN is NaN.
-        // Once the V tile has landed, the threads of those rows zero them.
+      const bool ragged = key_base / BKEYS == p_last / BKEYS && (p_last + 1) % BKEYS != 0;
+      // pages smaller than a tile: the window's first tile and the last tile of kept tokens may hold pages that were given back
+      const int walked = a.newest_first ? nt - 1 - j : j;
+      const bool holes = a.page_size < BKEYS && (walked == kept_tiles || walked + 1 == kept_tiles);
+      if (ragged || holes) {
+        // Value rows of positions past the portion's end hold whatever the page held before, and those of pages that
+        // were given back are any page's (another request's numbers, possibly not finite): P is zero there, but
+        // 0 x NaN is NaN. Once the V tile has landed, the threads of those rows zero them.
         if (!__all_sync(0xffffffffu, tc::mbar_wait(&v_full[sb], (j >> 1) & 1))) {
           if (lane == 0) atomicExch(a.status, 22);
           ok = false;
           break;
         }
-        if (r < BKEYS && key_base + r > p_last) {
+        if (r < BKEYS && (key_base + r > p_last ||
+                          (holes && a.block_table[(size_t)seq * a.table_stride + (key_base + r) / a.page_size] < 0))) {
           uint8_t* vrow = v_s + sb * KBYTES + (r / 8) * 1024 + (r % 8) * 128;
 #pragma unroll
           for (int blk = 0; blk < DBLK; ++blk)

@@ -33,6 +33,9 @@ class StepContext:
     # debug: choices a part is told to take instead of its own, by the name it reports them under
     # (the router's expert ids, int32 [N, k] in the step's flat token order)
     forced: Optional[Dict[str, torch.Tensor]] = None
+    # in front of the names that parts report and are told choices by, while a layer runs again: "run1/" in its
+    # second run (the model sets it; "" in the first)
+    run_prefix: str = ""
     # mixed steps only: flat rows of the requests that bring ONE token (int64 [D]) and the longest
     # context among them; None when the step is all portions or all single tokens
     decode_rows: Optional[torch.Tensor] = None

@@ -270,7 +270,7 @@ class SigmoidRoutedExperts(Part):
         if self.shared and self.OVERLAP_SHARED:
             shared, side = self._shared_on_side_stream(normed)
         router_in = normed if normed_f32 is None else normed_f32
-        forced = ctx.forced.get(f"{self.prefix}.router_ids") if ctx.forced else None
+        forced = ctx.forced.get(f"{ctx.run_prefix}{self.prefix}.router_ids") if ctx.forced else None
         if forced is None:
             ids, scores, plan = ops.router_plan(router_in, self.w_router, self.top_k, self.router_mode, self.score_scale,
                                                 bias=self.b_router)

@@ -112,9 +112,14 @@ class Model:
             else self.embedding.forward(ctx.tokens)
         if any(getattr(p, "needs_embedding_output", False) for p in self.interludes):
             ctx.scratch["embedding_output"] = residual.clone()       # the stream is summed into in place
-        pending = None
+        pending, tap, runs = None, ctx.tap, {}
         for entry in self.spec.schedule:
             layer = self.layers[entry.layer]
+            # what the parts of a layer report from its second run on carries the run's number
+            n = runs[entry.layer] = runs.get(entry.layer, -1) + 1
+            ctx.run_prefix = f"run{n}/" if n else ""
+            if tap is not None:
+                ctx.tap = tap if not n else (lambda name, t, prefix=ctx.run_prefix: tap(prefix + name, t))
             view = caches[entry.cache]
             if view.writes != entry.writes_cache:
                 view = CacheView(group=view.group, k_pages=view.k_pages, v_pages=view.v_pages, state=view.state,
@@ -122,6 +127,7 @@ class Model:
             if entry.interlude is not None:
                 residual, pending = self.interludes[entry.interlude].forward(residual, pending, ctx, entry.interlude_arg)
             residual, pending = layer.arrangement.forward(layer, residual, pending, ctx, view)
+        ctx.tap, ctx.run_prefix = tap, ""
         if logit_rows is None or logit_rows.numel() == 0:
             return None
         z = self.final_norm.forward(residual, pending, logit_rows)
