@@ -1417,6 +1417,206 @@ def case_bezasun_attention(tokens=2048, heads=16, reshaped=1):
     ops.check_tc_status()
 
 
+# --------------------------------------------------------------------------- Fofisun beside the closest existing models
+def _fofisun_config(width, heads, ff, layers, vocab=32000, window=4096):
+    """Differential attention on every layer (two maps of 64 over values of 128, a quarter as many key heads, four taps,
+    a window that keeps the first 4 tokens, an output gate); a dense feed-forward on every second layer and otherwise 8
+    clamped experts of half the dense size, 2 a token, with a gated shared expert of the same size."""
+    moe = {"kind": "moe", "expert": {"ff": ff // 2, "limit": 7.0}, "router": {"experts": 8, "top": 2}, "shared": {"ff": ff // 2, "limit": 7.0}}
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.5, "conv": 4,
+           "mask": {"size": window, "keep_first": 4}}
+    return {"architecture": "Fofisun", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+            "layers": [{"type": "attention", "mixer": att, "mlp": moe if i % 2 else {"kind": "dense", "ff": ff}} for i in range(layers)]}
+
+
+def case_fofisun(width=2048, heads=16, ff=8192, layers=6, tokens=2048, batch=8, context=4096):
+    """Prefill (one prompt of ``tokens`` in one step) and decode (``batch`` requests at ``context`` cached tokens,
+    captured steps) throughput of a Fofisun model with random weights beside Bezasun (the closest existing model:
+    attention on the same cache, experts with a shared one) and a dense Llama-4-shaped model of equal width, depth and
+    heads; then the new and the extended kernels alone beside their like kernels, with the bytes that must move over the
+    measured copy bandwidth. Markdown on standard output."""
+    import torch
+
+    from hi_b200.engine.core import Engine, StepEntry
+    from hi_b200.kernels import ops
+
+    pk = peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=DEV)
+    g = torch.Generator().manual_seed(0)
+
+    def timed(fn, reps=7, flush_l2=True):
+        fn()
+        ts = []
+        for _ in range(reps):
+            if flush_l2:
+                flush.zero_()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record(); fn(); b.record()
+            torch.cuda.synchronize()
+            ts.append(a.elapsed_time(b))
+        return sorted(ts)[len(ts) // 2]
+
+    print(f"peaks: {pk['hbm_gbs']:.0f} GB/s copy, {pk['bf16_tflops']:.0f} TFLOP/s bf16 ({pk['source']}); "
+          f"width {width}, {heads} heads, feed-forward {ff}, {layers} layers, bf16, random weights\n")
+    print("| model | prefill tokens/s | ms | decode tokens/s | ms/step | weights GB | launches/decode step |\n|---|---|---|---|---|---|---|")
+    for name, cfg in (("Fofisun", _fofisun_config(width, heads, ff, layers)), ("Bezasun", _bezasun_config(width, heads, ff, layers)),
+                      ("dense Llama-4 shape", _dense_llama_config(width, heads, ff, layers))):
+        eng = Engine.from_config(cfg, seed=0, dtype="bfloat16", device=DEV, kv_page_size=PAGE,
+                                 kv_cache_tokens=batch * (context + 256) + tokens + 256, max_active_requests=batch + 1)
+        vocab = eng.vocab_size
+        weights = sum(2 * int(torch.Size(sp.shape).numel()) for sp in eng.model.tensor_specs() if sp.init != "absent") / 1e9
+        prompt = torch.randint(0, vocab, (tokens,), generator=g).tolist()
+
+        def prefill():
+            eng.step([StepEntry("p", prompt, [tokens - 1])])
+            eng.finish("p")
+        t_pre = timed(prefill, reps=5)
+        for i in range(batch):
+            eng.assume_cached(i, context)
+        toks = torch.randint(0, vocab, (64, batch), generator=g).tolist()
+        turn = [0]
+
+        def decode():
+            eng.step([StepEntry(i, [toks[turn[0] % 64][i]], [0]) for i in range(batch)], borrow=True)
+            turn[0] += 1
+        for _ in range(4):
+            decode()
+        before = ops.LAUNCHES[0]
+        t_dec = timed(decode, reps=9, flush_l2=False)
+        launches = (ops.LAUNCHES[0] - before) // 10
+        print(f"| {name} | {tokens / t_pre * 1e3:,.0f} | {t_pre:.2f} | {batch / t_dec * 1e3:,.0f} | {t_dec:.3f} | {weights:.2f} | {launches} |")
+        del eng
+        torch.cuda.empty_cache()
+    rows = _fofisun_kernels(width, heads, ff, tokens, batch, context, timed, pk)
+    print("\n| step | kernel | us | MB that must move | GB/s | of the copy peak | |\n|---|---|---|---|---|---|---|")
+    print("\n".join(rows))
+
+
+def _fofisun_kernels(width, heads, ff, tokens, batch, context, timed, pk):
+    """The table rows of :func:`case_fofisun`: its kernels and their like kernels alone."""
+    import torch
+
+    from hi_b200.kernels import ops
+
+    bf, f32, dim, vdim, hd, taps = torch.bfloat16, torch.float32, 64, 128, 128, 4
+    dg = torch.Generator(device=DEV).manual_seed(0)
+    rnd = lambda *shape, dt=bf: torch.randn(*shape, device=DEV, generator=dg).to(dt)
+    rows, nkv, inter = [], max(1, heads // 4), ff // 2
+
+    def row(kind, name, ms, nbytes, note=""):
+        rows.append(f"| {kind} | {name} | {ms * 1e3:.1f} | {nbytes / 1e6:.1f} | {nbytes / ms / 1e6:,.0f} | "
+                    f"{nbytes / ms / 1e6 / pk['hbm_gbs']:.2f} | {note} |")
+
+    channels = (heads + nkv) * 2 * dim + nkv * vdim
+    for n, seqs, ctx_len, what in ((tokens, 1, tokens, "prefill"), (batch, batch, context, "decode")):
+        single = seqs == n
+        cu = torch.arange(0, n + 1, n // seqs, dtype=torch.int32, device=DEV)
+        sot = torch.repeat_interleave(torch.arange(seqs, device=DEV), n // seqs).to(torch.int32)
+        slots = torch.arange(seqs, dtype=torch.int32, device=DEV)
+        per = -(-ctx_len // PAGE)
+        pos = (torch.full((n,), ctx_len - 1, device=DEV) if single else torch.arange(n, device=DEV)).to(torch.int32)
+        table = torch.randperm(seqs * per, device=DEV, generator=dg).to(torch.int32).view(seqs, per).contiguous()
+        kp, vp = rnd(seqs * per, nkv, PAGE, hd), rnd(seqs * per, nkv, PAGE, hd)
+        # embedding, boundary
+        emb, tok = rnd(32000, width), torch.randint(0, 32000, (n,), device=DEV, generator=dg).to(torch.int32)
+        turns = torch.rand(width // 2, device=DEV, dtype=torch.float64)
+        row(what, "embedding + sinusoidal positions", timed(lambda: ops.embed_position(emb, tok, pos, turns)), n * width * 6)
+        row(what, "like: embedding", timed(lambda: ops.embed_gather(emb, tok)), n * width * 6)
+        x, d, w1, w2, wb = rnd(n, width, dt=f32), rnd(n, width), rnd(width, dt=f32), rnd(width, dt=f32), rnd(width)
+        routed, slot = rnd(2 * n, width, dt=f32), torch.randperm(2 * n, device=DEV, generator=dg).to(torch.int32)
+        rw = torch.rand(2 * n, device=DEV, generator=dg)
+        row(what, "boundary: norm of the result, sum, norm of the stream",
+            timed(lambda: ops.sandwich_step(x, w1, 1e-5, delta=d, weight=w2, eps=1e-5, out_dtype=bf)), n * width * 12)
+        row(what, "like: residual add + RMSNorm", timed(lambda: ops.add_rmsnorm(x, d, wb, 1e-5, bf)), n * width * 12)
+        row(what, "boundary with two routed rows a token and a float32 copy",
+            timed(lambda: ops.sandwich_step(x, w1, 1e-5, delta=d, routed=routed, slot_of_entry=slot, top_k=2, routed_weight=rw,
+                                            weight=w2, eps=1e-5, out_dtype=bf, also_f32=True)), n * width * 24)
+        row(what, "like: residual add + RMSNorm with the same",
+            timed(lambda: ops.add_rmsnorm(x, d, wb, 1e-5, bf, None, True, routed, slot, 2, rw)), n * width * 24)
+        # convolution, norms, append
+        proj, tw = rnd(n, channels + heads * vdim), rnd(taps, channels, dt=f32)
+        state, nw = torch.zeros(seqs, (taps - 1) * channels, device=DEV), rnd(dim, dt=f32)
+        conv = lambda: ops.conv_qkv(proj, tw, state, True, 1e-5, nw, nw, None, False, 1.0, pos, sot, cu, slots, table, kp, vp, True,
+                                    single, heads, nkv, 2, dim, vdim)
+        moved = n * (channels * 2 + (2 * heads + 2 * nkv) * hd * 2) + seqs * (taps - 1) * channels * 8
+        row(what, "q/k/v: convolution, norms, two maps, append (and its state)", timed(conv), moved)
+        qkv, nw2 = rnd(n, (heads + 2 * nkv) * hd), rnd(hd, dt=f32)
+        row(what, "like: q/k/v norms and append, one map, no convolution",
+            timed(lambda: ops.qkv_post(qkv, heads, nkv, hd, pos, None, False, True, 1e-5, None, sot, table, kp, vp, PAGE, True,
+                                       q_norm_weight=nw2, k_norm_weight=nw2, norm_first=True)), n * (heads + 2 * nkv) * hd * 4)
+        # attention: two maps with their finish, the same rows as plain softmax heads
+        q, gate = conv(), proj[:, channels:]
+        fin = (0.4, 1e-5, 0.5, vdim, gate)
+        plain_q = rnd(n, 2 * heads, hd)
+        pairs = n * ctx_len if single else n * (n + 1) // 2
+        kv = (n if single else 1) * ctx_len * nkv * hd * 4
+        tf = lambda ms, f: f"{pairs * heads * f / ms / 1e9:,.1f} TFLOP/s of its own products"
+        win = (context, 4) if single else (0, 0)
+        if single:
+            dec = lambda: ops.decode_attention(q, kp, vp, table, sot, pos, 0, win[0], dim ** -0.5, ctx_len, keep=win[1], parts=True)
+            pa, pm = dec()
+            ms = timed(dec)
+            row(what, f"two maps over a window with kept tokens: decode kernel ({pa.shape[2]} splits)", ms, kv + n * heads * hd * 4)
+            row(what, "merge of splits, difference, norm, gate",
+                timed(lambda: ops.diff_merge(pa, pm, *fin, torch.empty(n, heads * vdim, dtype=bf, device=DEV))), pa.numel() * 4 + n * heads * vdim * 4)
+            ms = timed(lambda: ops.decode_attention(plain_q, kp, vp, table, sot, pos, 0, 0, dim ** -0.5, ctx_len))
+            row(what, "like: plain softmax, decode kernel and merge (TMA tiles)", ms, kv + n * 2 * heads * hd * 4)
+            sl = torch.ones(2 * heads, device=DEV)
+            ms = timed(lambda: ops.decode_attention(plain_q, kp, vp, table, sot, pos, 0, 0, dim ** -0.5, ctx_len, slopes=sl))
+            row(what, "like: softmax with a distance bias, decode kernel and merge (cp.async tiles)", ms, kv + n * 2 * heads * hd * 4)
+        else:
+            ms = timed(lambda: ops.diff_prefill_attention_tc(q, kp, vp, table, cu, pos, 1, n, 0, 4096, 4, dim ** -0.5, *fin))
+            row(what, "two maps, difference, norm, gate in one kernel: tcgen05 prefill", ms, kv + n * heads * (2 * hd + 2 * vdim) * 2, tf(ms, 2 * 2 * (dim + vdim)))
+            ms = timed(lambda: ops.prefill_attention_tc(plain_q, kp, vp, table, cu, pos, 1, n, 0, 0, dim ** -0.5))
+            row(what, f"like: plain softmax of {2 * heads} heads of 128, tcgen05 prefill", ms, kv + n * 2 * heads * hd * 4, tf(ms, 2 * 2 * 2 * hd))
+            ms = timed(lambda: ops.prefill_attention_tc(plain_q[:, :heads].contiguous(), kp, vp, table, cu, pos, 1, n, 0, 0, dim ** -0.5))
+            row(what, f"like: plain softmax of {heads} heads of 128 (with the copy of its queries), tcgen05 prefill", ms, kv + n * heads * hd * 4, tf(ms, 2 * 2 * hd))
+            ms = timed(lambda: ops.diff_merge(*ops.prefill_attention(q, kp, vp, table, cu, pos, 1, n, 0, 4096, dim ** -0.5, keep=4, parts=True), *fin,
+                                              torch.empty(n, heads * vdim, dtype=bf, device=DEV)))
+            row(what, "two maps by the kernel of short portions (mma.sync) and the merge", ms, kv + n * heads * (2 * hd + 2 * vdim) * 2, tf(ms, 2 * 2 * (dim + vdim)))
+            ms = timed(lambda: ops.prefill_attention(plain_q, kp, vp, table, cu, pos, 1, n, 0, 0, dim ** -0.5))
+            row(what, f"like: plain softmax of {2 * heads} heads, mma.sync", ms, kv + n * 2 * heads * hd * 4, tf(ms, 2 * 2 * 2 * hd))
+        # feed-forward
+        z, zz = rnd(n, ff), rnd(n, 2 * inter + 8)
+        row(what, "exact gelu", timed(lambda: ops.gelu(z)), n * ff * 4)
+        row(what, "like: squared relu", timed(lambda: ops.relu2(z)), n * ff * 4)
+        row(what, "clamped unit with the token's gate (shared expert)", timed(lambda: ops.glu_limit(zz, inter, 7.0, 2 * inter)), n * inter * 6)
+        gu = zz[:, : 2 * inter].contiguous()
+        row(what, "like: SwiGLU", timed(lambda: ops.swiglu(gu)), n * inter * 6)
+        rx, rwt, rb = rnd(n, width, dt=f32), rnd(8, width), rnd(8, dt=f32)
+        row(what, "router with bias, softmax over the chosen, plan", timed(lambda: ops.router_plan(rx, rwt, 2, 3, bias=rb)), n * width * 4)
+        row(what, "like: sigmoid router, plan", timed(lambda: ops.router_plan(rx, rwt, 2)), n * width * 4)
+        _i, _s, plan = ops.router_plan(rx, rwt, 2, 3, bias=rb)
+        wg, wu, ones = rnd(8, inter, width), rnd(8, inter, width), torch.ones(n, 2, device=DEV)
+        xb = rx.to(bf)
+        for label, lim in (("experts' gate/up with the clamped unit, tcgen05", 7.0), ("like: with SwiGLU, tcgen05", 0.0)):
+            ms = timed(lambda: ops.moe_gate_up_tc(xb, plan, 2, wg, wu, ones, lim))
+            row(what, label, ms, 2 * wg.numel() * 2 + 2 * n * (2 * width + inter) * 2, f"{2 * n * 2 * inter * width * 2 / ms / 1e9:,.1f} TFLOP/s")
+    ops.check_tc_status()
+    return rows
+
+
+def case_fofisun_step(tokens=2048, batch=8, context=4096, width=2048, heads=16, ff=8192, layers=4):
+    """One Fofisun prompt step and two decode steps with every kernel launched on its own (no captured graph): for a
+    launch list under ncu."""
+    import torch
+
+    from hi_b200.engine.core import Engine, StepEntry
+
+    eng = Engine.from_config(_fofisun_config(width, heads, ff, layers), seed=0, dtype="bfloat16", device=DEV, kv_page_size=PAGE,
+                             kv_cache_tokens=batch * (context + 256) + tokens + 256, max_active_requests=batch + 1,
+                             use_cuda_graphs=False)
+    g = torch.Generator().manual_seed(0)
+    for rep in range(2):
+        eng.step([StepEntry("p", torch.randint(0, eng.vocab_size, (tokens,), generator=g).tolist(), [tokens - 1])])
+        eng.finish("p")
+    for i in range(batch):
+        eng.assume_cached(i, context)
+    for _ in range(3):
+        eng.step([StepEntry(i, [int(torch.randint(0, eng.vocab_size, (1,), generator=g))], [0]) for i in range(batch)])
+    torch.cuda.synchronize()
+
+
 # --------------------------------------------------------------------------- Fidatar beside the closest existing models
 def _fidatar_config(width, heads, ff, layers, vocab=32000, chunk=8192):
     """Layers in turn attention (heads of 128, a quarter as many key heads, chunks of 8,192, half of a head
@@ -1747,7 +1947,8 @@ CASES = {"sweep": case_sweep, "decode_timeline": case_decode_timeline, "prefill_
          "vinurax": case_vinurax, "delta_recurrence": case_delta_recurrence,
          "vinurax_step": case_vinurax_step, "fidatar": case_fidatar, "fidatar_step": case_fidatar_step,
          "mlstm_recurrence": case_mlstm_recurrence, "surinex": case_surinex, "surinex_step": case_surinex_step,
-         "bezasun": case_bezasun, "bezasun_step": case_bezasun_step, "bezasun_attention": case_bezasun_attention}
+         "bezasun": case_bezasun, "bezasun_step": case_bezasun_step, "bezasun_attention": case_bezasun_attention,
+         "fofisun": case_fofisun, "fofisun_step": case_fofisun_step}
 
 
 if __name__ == "__main__":

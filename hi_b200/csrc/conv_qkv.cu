@@ -19,7 +19,7 @@ namespace {
 struct ConvArgs {
   const void* proj;
   long long ld;                  // elements between rows of proj
-  const float* taps;             // [channels][K], or null (K == 1: no convolution)
+  const float* taps;             // [K][channels], or null (K == 1: no convolution)
   float* state;                  // [slots][state_stride], the K - 1 rows of a request at conv_off
   long long state_stride, conv_off;
   const float* q_w;
@@ -55,11 +55,29 @@ __device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) {
   *reinterpret_cast<uint4*>(p) = pack;
 }
 
-constexpr int kThreads = 256;
+// 8 consecutive elements as they lie in memory
+template <typename T> struct Raw8 { uint4 w[sizeof(T) / 2]; };
+template <typename T> __device__ __forceinline__ Raw8<T> raw8(const T* p) {
+  Raw8<T> r;
+#pragma unroll
+  for (int i = 0; i < (int)(sizeof(T) / 2); ++i) r.w[i] = reinterpret_cast<const uint4*>(p)[i];
+  return r;
+}
+__device__ __forceinline__ float element(const Raw8<float>& r, int e) {
+  const uint4 q = r.w[e / 4];
+  return __uint_as_float(e % 4 == 0 ? q.x : e % 4 == 1 ? q.y : e % 4 == 2 ? q.z : q.w);
+}
+__device__ __forceinline__ float element(const Raw8<__nv_bfloat16>& r, int e) {
+  const uint4 q = r.w[0];
+  const uint32_t w = e / 2 == 0 ? q.x : e / 2 == 1 ? q.y : e / 2 == 2 ? q.z : q.w;
+  return __uint_as_float(e % 2 ? w & 0xffff0000u : w << 16);
+}
+
+constexpr int kThreads = 128;
 
 // A vector (a head's query or key of one map, or a value) is taken by `lanes` neighbouring lanes (a power of two) of 8
-// channels each; a thread goes over kRun consecutive rows of the step, its channels' taps read once and a request's
-// rows sliding through a window of K registers a channel. Blocks y < qk_blocks take query and key vectors, the rest
+// channels each; a thread goes over kRun consecutive rows of the step, its channels' taps read once. A run inside one
+// request, behind its first K - 1 rows, has all its rows asked for at once; others slide a window of K registers a channel. Blocks y < qk_blocks take query and key vectors, the rest
 // value vectors (which may be of another size).
 template <typename T, int K, int kRun>
 __global__ void __launch_bounds__(kThreads) conv_qkv_kernel(const ConvArgs a, int qk_blocks, int qk_lanes, int v_lanes) {
@@ -78,24 +96,82 @@ __global__ void __launch_bounds__(kThreads) conv_qkv_kernel(const ConvArgs a, in
   const T* proj = reinterpret_cast<const T*>(a.proj);
   float w[8 * K], nw[8];
 #pragma unroll
-  for (int i = 0; i < 8 * K; ++i) w[i] = 1.f;
+  for (int i = 0; i < 8 * K; ++i) w[i] = 1.f;                                  // [tap][channel]
   if (owns && a.taps) {
 #pragma unroll
-    for (int i = 0; i < 2 * K; ++i) {
-      const float4 f = *reinterpret_cast<const float4*>(a.taps + (size_t)c0 * K + 4 * i);
-      w[4 * i] = f.x; w[4 * i + 1] = f.y; w[4 * i + 2] = f.z; w[4 * i + 3] = f.w;
-    }
+    for (int j = 0; j < K; ++j)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const float4 f = *reinterpret_cast<const float4*>(a.taps + (size_t)j * channels + c0 + 4 * i);
+        w[8 * j + 4 * i] = f.x; w[8 * j + 4 * i + 1] = f.y; w[8 * j + 4 * i + 2] = f.z; w[8 * j + 4 * i + 3] = f.w;
+      }
   }
   const float* norm_w = is_v ? nullptr : (is_q ? a.q_w : a.k_w);
 #pragma unroll
   for (int e = 0; e < 8; ++e) nw[e] = owns && norm_w ? norm_w[sub * 8 + e] : 1.f;
   const int map = is_v ? 0 : (is_q ? vec : vec - nq) % a.maps;
   const int own_at = map * a.dim;                                              // (values: 0)
+  // one row's vector: norm, place in its row of q or of the cache
+  auto finish = [&](float (&y)[8], float ss, int t, int s, int pos) {
+    if (!is_v && a.norm) {                                                     // the same for the whole block
+      for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float inv = rsqrtf(ss / (float)size + a.eps);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] *= inv * nw[e];
+    }
+    if (!exists) return;
+    T* row;
+    if (is_q) {
+      row = reinterpret_cast<T*>(a.q_out) + ((size_t)t * nq + vec) * a.hd;
+    } else {
+      const int page = a.block_table[(size_t)s * a.table_stride + pos / a.page_size];
+      if (page < 0) return;                                                    // the host reserves pages before the step
+      const int kvh = is_v ? vec : (vec - nq) / a.maps;
+      row = reinterpret_cast<T*>(is_v ? a.v_pages : a.k_pages) +
+            (((size_t)page * a.kv_heads + kvh) * a.page_size + pos % a.page_size) * a.hd;
+    }
+    if (owns) store8(row + own_at + sub * 8, y);
+    const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (is_q && owns)
+      for (int m = 0; m < a.maps; ++m)
+        if (m != map) store8(row + m * a.dim + sub * 8, zero);
+    if (is_q || map == 0)                                                      // padding behind the maps (or the value)
+      for (int d = (is_v ? a.vdim : a.maps * a.dim) + sub * 8; d < a.hd; d += lanes * 8) store8(row + d, zero);
+  };
+  const int t0 = blockIdx.x * kRun;
+  if constexpr (kRun > 1) {
+    const int s = a.seq_of_token[t0];
+    if (t0 + kRun <= a.n_tokens && t0 - a.cu_seqlens[s] >= K - 1 && t0 + kRun <= a.cu_seqlens[s + 1]) {
+      Raw8<T> rows[kRun + K - 1];
+      if (owns) {
+#pragma unroll
+        for (int i = 0; i < kRun + K - 1; ++i) rows[i] = raw8(proj + (size_t)(t0 - (K - 1) + i) * a.ld + c0);
+      }
+      const int pos0 = a.positions[t0];
+#pragma unroll
+      for (int i = 0; i < kRun; ++i) {
+        float y[8];
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          float acc = 0.f;
+          if (owns) {
+#pragma unroll
+            for (int j = 0; j < K; ++j) acc = fmaf(w[8 * j + e], element(rows[i + j], e), acc);
+          }
+          y[e] = acc;
+          ss += acc * acc;
+        }
+        finish(y, ss, t0 + i, s, pos0 + i);
+      }
+      return;
+    }
+  }
   float x[K][8];
   int prev_seq = -1;
 #pragma unroll 1
   for (int i = 0; i < kRun; ++i) {
-    const int t = blockIdx.x * kRun + i;
+    const int t = t0 + i;
     if (t >= a.n_tokens) break;                                                // the same for the whole block
     const int s = a.seq_of_token[t];
     if (owns) {
@@ -124,36 +200,12 @@ __global__ void __launch_bounds__(kThreads) conv_qkv_kernel(const ConvArgs a, in
       float acc = 0.f;
       if (owns) {
 #pragma unroll
-        for (int j = 0; j < K; ++j) acc = fmaf(w[e * K + j], x[j][e], acc);
+        for (int j = 0; j < K; ++j) acc = fmaf(w[8 * j + e], x[j][e], acc);
       }
       y[e] = acc;
       ss += acc * acc;
     }
-    if (!is_v && a.norm) {                                                     // the same for the whole block
-      for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      const float inv = rsqrtf(ss / (float)size + a.eps);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) y[e] *= inv * nw[e];
-    }
-    if (!exists) continue;
-    T* row;
-    const int pos = a.positions[t];
-    if (is_q) {
-      row = reinterpret_cast<T*>(a.q_out) + ((size_t)t * nq + vec) * a.hd;
-    } else {
-      const int page = a.block_table[(size_t)s * a.table_stride + pos / a.page_size];
-      if (page < 0) continue;                                                  // the host reserves pages before the step
-      const int kvh = is_v ? vec : (vec - nq) / a.maps;
-      row = reinterpret_cast<T*>(is_v ? a.v_pages : a.k_pages) +
-            (((size_t)page * a.kv_heads + kvh) * a.page_size + pos % a.page_size) * a.hd;
-    }
-    if (owns) store8(row + own_at + sub * 8, y);
-    const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    if (is_q && owns)
-      for (int m = 0; m < a.maps; ++m)
-        if (m != map) store8(row + m * a.dim + sub * 8, zero);
-    if (is_q || map == 0)                                                      // padding behind the maps (or the value)
-      for (int d = (is_v ? a.vdim : a.maps * a.dim) + sub * 8; d < a.hd; d += lanes * 8) store8(row + d, zero);
+    finish(y, ss, t, s, a.positions[t]);
     // the request's only token of the step: its inputs move up a row in the state, which this thread alone reads and
     // writes at these channels
     if (K > 1 && a.fuse_tail && owns) {
@@ -210,7 +262,7 @@ __global__ void conv_qkv_general_kernel(const ConvArgs a) {
           const int rel = local - (a.K - 1) + j;
           const float u = rel >= 0 ? hb::to_f32(proj[(size_t)(start + rel) * a.ld + c0 + d])
                                    : tail[(size_t)(a.K - 1 + rel) * channels + c0 + d];
-          acc = fmaf(a.taps[(size_t)(c0 + d) * a.K + j], u, acc);
+          acc = fmaf(a.taps[(size_t)j * channels + c0 + d], u, acc);
         }
       } else {
         acc = hb::to_f32(proj[(size_t)t * a.ld + c0 + d]);
@@ -291,7 +343,7 @@ int launch_conv(const ConvArgs& a, bool fast, cudaStream_t stream) {
 
 }  // namespace
 
-// `taps` [channels][taps_n] float32 or null (no convolution; taps_n is then 1). `single_tokens`: every request of the
+// `taps` [taps_n][channels] float32 or null (no convolution; taps_n is then 1). `single_tokens`: every request of the
 // step brings one token. `moved` (host, one int): set to 1 when the kernel moved the requests' inputs in the state
 // itself, 0 when the caller has to (hb_delta_conv_update has the state layout's rule).
 extern "C" int hb_conv_qkv(const void* proj, int dtype, long long ld, const float* taps, int taps_n, float* state,

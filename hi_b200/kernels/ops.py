@@ -1519,7 +1519,7 @@ def conv_qkv(proj: torch.Tensor, taps: Optional[torch.Tensor], state: Optional[t
              maps: int, dim: int, vdim: int) -> torch.Tensor:
     """Short causal convolution over time of the projected channels, RMS norm of q and k per vector, rotation, cache
     append. ``proj`` [N, >= channels] has the unpadded rows [q: heads * maps * dim | k: kv_heads * maps * dim |
-    v: kv_heads * vdim | ...]; ``taps`` float32 [channels, K] or None; ``state`` float32 [slots, (K - 1) * channels] is
+    v: kv_heads * vdim | ...]; ``taps`` float32 [K, channels] or None; ``state`` float32 [slots, (K - 1) * channels] is
     read and moved on. Returns q [N, heads * maps, hd] with hd the pages' row length: a map's query at its place of the
     row, zeros elsewhere; key rows are [map 1 | map 2 | zeros], value rows [vdim | zeros]."""
     if not proj.is_cuda or proj.dim() != 2 or proj.stride(1) != 1:
@@ -1536,9 +1536,9 @@ def conv_qkv(proj: torch.Tensor, taps: Optional[torch.Tensor], state: Optional[t
     taps_n, state_stride = 1, 0
     if taps is not None:
         _need(taps, "taps", torch.float32)
-        taps_n = taps.shape[1]
-        if taps.shape[0] != channels:
-            raise KernelError(f"taps for {taps.shape[0]} channels, the projection has {channels}")
+        taps_n = taps.shape[0]
+        if taps.shape[1] != channels:
+            raise KernelError(f"taps for {taps.shape[1]} channels, the projection has {channels}")
         if taps_n > 1:
             _need(state, "state", torch.float32)
             state_stride = state.shape[1]

@@ -349,7 +349,7 @@ class AttentionMixer(Part):
         if self.norm_weighted:
             self.w_qnorm, self.w_knorm = (fetch(f"{self.prefix}.{n}.norm").to(f32).contiguous() for n in "qk")
         if self.taps:
-            self.conv_taps = torch.cat([fetch(f"{self.prefix}.{n}.conv").to(f32) for n in "qkv"], dim=0).contiguous()
+            self.conv_taps = torch.cat([fetch(f"{self.prefix}.{n}.conv").to(f32) for n in "qkv"], dim=0).t().contiguous()      # [K, channels]
         if self.diff is not None:
             lq1, lk1, lq2, lk2 = (fetch(f"{self.prefix}.{n}").to(torch.float64) for n in ("lq1", "lk1", "lq2", "lk2"))
             self.lam = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum()) + self.diff)

@@ -162,7 +162,7 @@ def test_conv_qkv(dt, tol, heads, kvh, maps, dim, vdim, hd, taps, rot):
         sot = torch.cat([torch.full((n,), i) for i, (_s, n) in enumerate(step)]).to(torch.int32).to(DEV)
         cu = torch.tensor([0] + torch.tensor([n for _s, n in step]).cumsum(0).tolist(), dtype=torch.int32, device=DEV)
         sl = torch.tensor([slots[s] for s in seqs], dtype=torch.int32, device=DEV)
-        q = o.conv_qkv(x, None if w is None else w.to(DEV), state, True, 1e-5, qn.to(DEV), kn.to(DEV),
+        q = o.conv_qkv(x, None if w is None else w.t().contiguous().to(DEV), state, True, 1e-5, qn.to(DEV), kn.to(DEV),
                        None if inv is None else inv.to(DEV), bool(rot and rot[1]), 1.2 if rot else 1.0, pos, sot, cu, sl,
                        table[seqs].contiguous().to(DEV), k_pages, v_pages, True, all(n == 1 for _s, n in step), heads, kvh, maps,
                        dim, vdim)
