@@ -200,8 +200,8 @@ class AttentionMixer(Part):
       ``conv``         None | K: every channel of q, k and v passes a causal convolution of K taps over time right
                        after the projection, y_t = sum_j taps[:, j] u_(t - K + 1 + j) (zeros before the start):
                        ``<prefix>.{q,k,v}.conv`` [channels, K]; the last K - 1 inputs are state of the request
-      ``differential``  None | c: every query and key head has two maps of ``head_dim`` (projection rows head by head
-                       [map 1, map 2]), each an attention of its own over the same values; their results a1, a2 give
+      ``differential``  None | c: every query and key head has two maps of ``head_dim`` (a head's second map
+                       follows its first in the projection's rows), each an attention of its own over the same values; their results a1, a2 give
                        o = a1 - lambda a2 with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + c (one number a layer,
                        ``<prefix>.lq1|lk1|lq2|lk2`` [head_dim]), and o <- o / rms(o) (over the head's values, eps
                        ``qk_norm_eps``) * (1 - c)
