@@ -33,7 +33,7 @@ import os
 import sys
 
 PAGE_SIZE = 64
-MAX_LIVE_REQUESTS = 8
+MAX_LIVE_REQUESTS = 4
 PAGE_SIZES = (8, 16, 32, 64, 128)      # the reference's page sizes and one larger (crates/hi-cuda/src/lib.rs:634-636)
 
 
