@@ -5,6 +5,7 @@ architecture is added the same way from anywhere: a typed config reader, a build
 ``model_type`` names (the reference routes ``llama4`` / ``llama4_text`` to its Llama 4 model:
 crates/hi-mlx/src/config.rs:620-637, crates/hi-mlx/src/models.rs:373-375)."""
 from .config import bezasun as _bezasun
+from .config import darotar as _darotar
 from .config import fidatar as _fidatar
 from .config import fofisun as _fofisun
 from .config import surinex as _surinex
@@ -12,6 +13,7 @@ from .config import vinurax as _vinurax
 from .config.llama4 import Llama4TextConfig
 from .config.registry import Architecture, register_architecture
 from .parts.bezasun import build_bezasun_spec, normalize_bezasun_tensor_name
+from .parts.darotar import build_darotar_spec, normalize_darotar_tensor_name
 from .parts.fidatar import build_fidatar_spec, normalize_fidatar_tensor_name
 from .parts.fofisun import build_fofisun_spec, normalize_fofisun_tensor_name
 from .parts.llama4 import build_llama4_spec, derive_llama4_tensors, normalize_llama4_tensor_name
@@ -47,3 +49,8 @@ register_architecture(
     ["Fofisun", "fofisun"],
     Architecture(name="fofisun", parse_config=_fofisun.FofisunConfig.from_json, build_spec=build_fofisun_spec,
                  normalize_tensor_name=normalize_fofisun_tensor_name))
+
+register_architecture(
+    ["Darotar", "darotar"],
+    Architecture(name="darotar", parse_config=_darotar.DarotarConfig.from_json, build_spec=build_darotar_spec,
+                 normalize_tensor_name=normalize_darotar_tensor_name, sizes_from_tensors=_darotar.sizes_from_tensors))

@@ -39,7 +39,7 @@ int hb_moe_combine(const float* y, const int* slot_of_entry, const float* routed
 int hb_qkv_post(const void* qkv, int dtype, const float* inv_freq, int rot_pairs, int interleaved, int qk_norm,
                 float qk_eps, int temp_on, float floor_scale, float attn_scale, const float* q_norm_w,
                 const float* k_norm_w, int norm_first, int norm_dim, float rot_mul, const float* v_inv_freq,
-                int v_pairs, int v_interleaved, const int* positions,
+                int v_pairs, int v_interleaved, int v_is_k, const int* positions,
                 const int* seq_of_token, const int* block_table, int table_stride, void* q_out, void* k_pages,
                 void* v_pages, int page_size, int write_kv, int n_tokens, int nh, int nkv, int hd,
                 cudaStream_t stream);
@@ -82,7 +82,7 @@ int hb_attention_decode_fused(const void* qkv, const float* inv_freq, int rot_pa
                               int hd, int page_size, int chunk, int window, float scale, int split_size,
                               int max_splits, float* part_acc, float* part_ml, int* counters, int* status,
                               const float* q_norm_w, const float* k_norm_w, int norm_first, float rot_mul, int sink,
-                              cudaStream_t stream);
+                              int v_is_k, cudaStream_t stream);
 
 // hb_attention_prefill with reshaped scores: softcap, slopes, sink_values as hb_paged_attention
 int hb_attention_prefill_reshaped(const void* q, const void* k_pages, const void* v_pages, const int* block_table,

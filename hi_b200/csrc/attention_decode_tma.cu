@@ -55,7 +55,7 @@ struct Args {
 
 // What the fused form needs beside Args.
 struct Fuse {
-  const __nv_bfloat16* qkv;      // [n_tokens, (nh + 2 nkv) * head_dim]: q heads, k heads, v heads
+  const __nv_bfloat16* qkv;      // [n_tokens, (nh + 2 nkv) * head_dim]: q heads, k heads, v heads (none with v_is_k)
   const float* inv_freq;         // [rot_pairs], or null: no rotation
   int rot_pairs;                 // the first 2 * rot_pairs dims of a head rotate (a multiple of 8 pairs)
   __nv_bfloat16* k_pages;
@@ -69,6 +69,7 @@ struct Fuse {
   const float* k_w;
   int norm_first;
   float rot_mul;
+  int v_is_k;                    // a row of qkv has no v heads: the key as projected is the value
 };
 
 // One head of the q/k/v row as qkv_post.cu encodes it: head_dim / 16 neighbouring lanes, each with
@@ -253,7 +254,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     for (int c = tid; c < (ROWS - G) * CHUNKS; c += NWARPS * 32)      // the tile's rows past the group are zeros
       *reinterpret_cast<uint4*>(q_s + (G + c / CHUNKS) * STRIDE + (c % CHUNKS) * 8) = make_uint4(0u, 0u, 0u, 0u);
     __syncthreads();                               // sines and cosines; the barriers are initialised
-    const __nv_bfloat16* row = f.qkv + (size_t)t * (a.nh + 2 * a.nkv) * HD;
+    const __nv_bfloat16* row = f.qkv + (size_t)t * (a.nh + (f.v_is_k ? 1 : 2) * a.nkv) * HD;
     const int sub = lane % LPH, slot = warp * HPW + lane / LPH;     // NWARPS * HPW = 16 head slots
     {
       const bool active = slot < G;
@@ -268,7 +269,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     if (last == pos && warp == 0) {                // this block's range ends at the token itself: its key and value
       const bool active = slot < 2;
       const int kind = 1 + (slot & 1);
-      const __nv_bfloat16* src = row + (size_t)(a.nh + (kind == 2 ? a.nkv : 0) + kvh) * HD;
+      const __nv_bfloat16* src = row + (size_t)(a.nh + (kind == 2 && !f.v_is_k ? a.nkv : 0) + kvh) * HD;
       encode_head<HD>(src, kind, active, sub, f, cs_s, sn_s, pos, own_c0, own_c1, own_d0, own_d1);
       own_kv = active;
       const int page = table[pos / a.page_size];
@@ -594,7 +595,7 @@ extern "C" int hb_attention_decode_tma(const void* q, const void* k_pages, const
 // The fused form: `qkv` [n_tokens, (nh + 2 nkv) * hd] is the q/k/v projection's output; the kernel
 // encodes q, k and v as hb_qkv_post does (inv_freq [rot_pairs] or null; pairs (j, j + rot_pairs) or
 // (2j, 2j + 1); weightless norm after the rotation, or with norm_first the weighted RMS norm before it; rot_mul on
-// cos and sin; temperature on q; sink: one more term of score 0 in the softmax's denominator), appends the token's key and value to its page,
+// cos and sin; temperature on q; v_is_k as in hb_qkv_post; sink: one more term of score 0 in the softmax's denominator), appends the token's key and value to its page,
 // attends, and combines its own splits: `counters` holds n_tokens * nkv ints that are zero before
 // the call and zero after it. With `counters` null the splits are left in part_acc / part_ml for
 // hb_attention_merge, as hb_attention_decode_tma leaves them. Same shapes and refusals as hb_attention_decode_tma; every token is
@@ -606,7 +607,7 @@ extern "C" int hb_attention_decode_fused(const void* qkv, const float* inv_freq,
                                          int nh, int nkv, int hd, int page_size, int chunk, int window, float scale,
                                          int split_size, int max_splits, float* part_acc, float* part_ml,
                                          int* counters, int* status, const float* q_norm_w, const float* k_norm_w,
-                                         int norm_first, float rot_mul, int sink, cudaStream_t stream) {
+                                         int norm_first, float rot_mul, int sink, int v_is_k, cudaStream_t stream) {
   if (!qkv || !k_pages || !v_pages || !block_table || !seq_of_token || !positions || !out || !status) return HB_ERR_BAD_ARG;
   if (n_tokens < 0 || n_pages <= 0 || nh <= 0 || nkv <= 0 || nh % nkv != 0 || page_size <= 0 || table_stride <= 0 ||
       chunk < 0 || window < 0 || max_splits < 1 || split_size <= 0 || split_size % TILE != 0)
@@ -624,7 +625,7 @@ extern "C" int hb_attention_decode_fused(const void* qkv, const float* inv_freq,
          table_stride, nh, nkv, page_size, chunk, split_size, max_splits, page_size < TILE ? page_size : TILE, scale, sink};
   if (!norm_first && (q_norm_w || k_norm_w || rot_mul != 1.f)) return HB_ERR_UNSUPPORTED;   // as hb_qkv_post
   Fuse f{(const __nv_bfloat16*)qkv, inv_freq, rot_pairs, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, counters,
-         interleaved, qk_norm, temp_on, qk_eps, floor_scale, attn_scale, q_norm_w, k_norm_w, norm_first, rot_mul};
+         interleaved, qk_norm, temp_on, qk_eps, floor_scale, attn_scale, q_norm_w, k_norm_w, norm_first, rot_mul, v_is_k};
   if (hd == 128) return launch<128, true>(k_pages, v_pages, n_pages, n_tokens, a, f, stream);
   if (hd == 64) return launch<64, true>(k_pages, v_pages, n_pages, n_tokens, a, f, stream);
   return HB_ERR_UNSUPPORTED;

@@ -40,11 +40,12 @@ __device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) {
 // computes the token's sines and cosines once.
 // norm_first: the norm of q and k is an RMS norm over the head BEFORE the rotation, with a weight per dim
 // (q_w / k_w, float32 [hd], or null); rot_mul multiplies cos and sin.
+// v_is_k: a row of qkv has q and k heads only; a key head as projected, before norm and rotation, is the value too.
 template <typename T>
 __global__ void qkv_post_kernel(const T* __restrict__ qkv, const float* __restrict__ inv_freq,
                                 int rot_pairs, int interleaved, int qk_norm, float qk_eps, int temp_on,
                                 float floor_scale, float attn_scale, const float* __restrict__ q_w,
-                                const float* __restrict__ k_w, int norm_first, float rot_mul,
+                                const float* __restrict__ k_w, int norm_first, float rot_mul, int v_is_k,
                                 const int* __restrict__ positions,
                                 const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
                                 int table_stride, T* __restrict__ q_out, T* __restrict__ k_pages,
@@ -52,7 +53,7 @@ __global__ void qkv_post_kernel(const T* __restrict__ qkv, const float* __restri
                                 int nkv, int hd, int lanes_per_head) {
   __shared__ float cs_s[kMaxHeadDim / 2], sn_s[kMaxHeadDim / 2];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int heads_total = nh + 2 * nkv;
+  const int heads_total = nh + (v_is_k ? 1 : 2) * nkv;
   const int heads_per_warp = 32 / lanes_per_head;
   const int t = blockIdx.x;
   const int first_head = blockIdx.y * kWarpsPerBlock * heads_per_warp;
@@ -72,6 +73,7 @@ __global__ void qkv_post_kernel(const T* __restrict__ qkv, const float* __restri
   const int kind = head < nh ? 0 : (head < nh + nkv ? 1 : 2);  // q, k, v
   bool active = head < heads_total && sub * 16 < hd && (kind == 0 || write_kv);
   T* dst = nullptr;
+  T* raw_dst = nullptr;                                  // v_is_k: where a key head's projection goes as a value
   if (active) {
     if (kind == 0) {
       dst = q_out + ((size_t)t * nh + head) * hd;
@@ -81,7 +83,9 @@ __global__ void qkv_post_kernel(const T* __restrict__ qkv, const float* __restri
       active = page >= 0;    // the host reserves pages before the step; without one there is nothing to write into
       const int kvh = kind == 1 ? head - nh : head - nh - nkv;
       T* pool = kind == 1 ? k_pages : v_pages;
-      dst = pool + (((size_t)(active ? page : 0) * nkv + kvh) * page_size + (pos % page_size)) * hd;
+      const size_t at = (((size_t)(active ? page : 0) * nkv + kvh) * page_size + (pos % page_size)) * hd;
+      dst = pool + at;
+      if (v_is_k) raw_dst = v_pages + at;
     }
   }
   const int j0 = sub * 8;                                // pairs j0 .. j0 + 7
@@ -103,6 +107,14 @@ __global__ void qkv_post_kernel(const T* __restrict__ qkv, const float* __restri
     } else {
       hb::load8(src + j0, a);
       hb::load8(src + half + j0, b);
+    }
+    if (raw_dst != nullptr) {
+      const uint4* from0 = reinterpret_cast<const uint4*>(src + (consecutive ? 2 * j0 : j0));
+      const uint4* from1 = reinterpret_cast<const uint4*>(src + (consecutive ? 2 * j0 + 8 : half + j0));
+      uint4* to0 = reinterpret_cast<uint4*>(raw_dst + (consecutive ? 2 * j0 : j0));
+      uint4* to1 = reinterpret_cast<uint4*>(raw_dst + (consecutive ? 2 * j0 + 8 : half + j0));
+#pragma unroll
+      for (int i = 0; i < (int)sizeof(T) / 2; ++i) { to0[i] = from0[i]; to1[i] = from1[i]; }
     }
   }
   if (norm_first) {
@@ -172,7 +184,7 @@ __global__ void qkv_post_general_kernel(const T* __restrict__ qkv, const float* 
                                         int interleaved, int qk_norm, float qk_eps, int temp_on, float floor_scale,
                                         float attn_scale, const float* __restrict__ q_w, const float* __restrict__ k_w,
                                         int norm_first, int norm_dim, float rot_mul,
-                                        const float* __restrict__ v_inv_freq, int v_pairs, int v_interleaved,
+                                        const float* __restrict__ v_inv_freq, int v_pairs, int v_interleaved, int v_is_k,
                                         const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                                         const int* __restrict__ block_table, int table_stride, T* __restrict__ q_out,
                                         T* __restrict__ k_pages, T* __restrict__ v_pages, int page_size, int write_kv,
@@ -195,19 +207,22 @@ __global__ void qkv_post_general_kernel(const T* __restrict__ qkv, const float* 
   if (write_kv)
     for (int j = threadIdx.x; j < v_pairs; j += blockDim.x) sincosf((float)pos * v_inv_freq[j], &vsn[j], &vcs[j]);
   __syncthreads();
-  const int heads_total = nh + 2 * nkv;
+  const int heads_total = nh + (v_is_k ? 1 : 2) * nkv;
   const int rot = 2 * rot_pairs;
   for (int head = warp; head < heads_total; head += nwarps) {
     const int kind = head < nh ? 0 : (head < nh + nkv ? 1 : 2);
     if (kind != 0 && !write_kv) break;          // heads are ordered q, k, v
     T* dst;
+    T* raw_dst = nullptr;                       // v_is_k: where a key head's projection goes as a value
     if (kind == 0) {
       dst = q_out + ((size_t)t * nh + head) * hd;
     } else {
       const int page = block_table[(size_t)seq_of_token[t] * table_stride + pos / page_size];
       if (page < 0) continue;                   // the host reserves pages before the step
       const int kvh = kind == 1 ? head - nh : head - nh - nkv;
-      dst = (kind == 1 ? k_pages : v_pages) + (((size_t)page * nkv + kvh) * page_size + (pos % page_size)) * hd;
+      const size_t at = (((size_t)page * nkv + kvh) * page_size + (pos % page_size)) * hd;
+      dst = (kind == 1 ? k_pages : v_pages) + at;
+      if (v_is_k) raw_dst = v_pages + at;
     }
     const T* src = qkv + ((size_t)t * heads_total + head) * hd;
     if (kind == 2) {
@@ -239,6 +254,7 @@ __global__ void qkv_post_general_kernel(const T* __restrict__ qkv, const float* 
     for (int d = lane; d < hd; d += 32) {
       const float x = hb::to_f32(src[d]);
       row[d] = x;
+      if (raw_dst != nullptr) raw_dst[d] = src[d];
       if (d < norm_dim) ss += x * x;
     }
     ss = hb::warp_sum(ss);
@@ -275,7 +291,7 @@ __global__ void qkv_post_general_kernel(const T* __restrict__ qkv, const float* 
 extern "C" int hb_qkv_post(const void* qkv, int dtype, const float* inv_freq, int rot_pairs, int interleaved,
                            int qk_norm, float qk_eps, int temp_on, float floor_scale, float attn_scale,
                            const float* q_norm_w, const float* k_norm_w, int norm_first, int norm_dim, float rot_mul,
-                           const float* v_inv_freq, int v_pairs, int v_interleaved,
+                           const float* v_inv_freq, int v_pairs, int v_interleaved, int v_is_k,
                            const int* positions, const int* seq_of_token, const int* block_table,
                            int table_stride, void* q_out, void* k_pages, void* v_pages, int page_size,
                            int write_kv, int n_tokens, int nh, int nkv, int hd, cudaStream_t stream) {
@@ -288,21 +304,21 @@ extern "C" int hb_qkv_post(const void* qkv, int dtype, const float* inv_freq, in
   if (norm_dim <= 0) norm_dim = hd;
   if (norm_dim > hd || 2 * rot_pairs > norm_dim) return HB_ERR_BAD_ARG;
   if (!v_inv_freq) v_pairs = 0;
-  if (v_pairs < 0 || 2 * v_pairs > hd) return HB_ERR_BAD_ARG;
+  if (v_pairs < 0 || 2 * v_pairs > hd || (v_is_k && v_pairs > 0)) return HB_ERR_BAD_ARG;
   if (n_tokens == 0) return HB_OK;
   const bool fast = v_pairs == 0 && hd % 16 == 0 && hd <= kMaxHeadDim && rot_pairs % 8 == 0 /* whole lanes rotate */ && norm_dim == hd &&
                     (norm_first || (!q_norm_w && !k_norm_w && rot_mul == 1.f));
   if (!fast) {
     // a norm after a rotation that changes lengths would need the rotated squares; no model asks for it
     if (qk_norm && !norm_first && (rot_mul != 1.f || q_norm_w || k_norm_w)) return HB_ERR_UNSUPPORTED;
-    const int heads_all = nh + 2 * nkv;
+    const int heads_all = nh + (v_is_k ? 1 : 2) * nkv;
     const int warps = heads_all < 8 ? heads_all : 8;
     const size_t smem = (size_t)(2 * rot_pairs + 2 * v_pairs + warps * hd) * sizeof(float);
     if (smem > 48 * 1024) return HB_ERR_UNSUPPORTED;
 #define HB_QKV_GENERAL(T)                                                                                          \
     qkv_post_general_kernel<T><<<n_tokens, warps * 32, smem, stream>>>(                                             \
         (const T*)qkv, inv_freq, rot_pairs, interleaved, qk_norm, qk_eps, temp_on, floor_scale, attn_scale, q_norm_w, \
-        k_norm_w, norm_first, norm_dim, rot_mul, v_inv_freq, v_pairs, v_interleaved, positions, seq_of_token,       \
+        k_norm_w, norm_first, norm_dim, rot_mul, v_inv_freq, v_pairs, v_interleaved, v_is_k, positions, seq_of_token, \
         block_table, table_stride, (T*)q_out,                                                                       \
         (T*)k_pages, (T*)v_pages, page_size, write_kv, nh, nkv, hd)
     if (dtype == HB_DTYPE_F32) HB_QKV_GENERAL(float);
@@ -312,7 +328,7 @@ extern "C" int hb_qkv_post(const void* qkv, int dtype, const float* inv_freq, in
     HB_LAUNCH_CHECK();
     return HB_OK;
   }
-  const int heads_total = nh + 2 * nkv;
+  const int heads_total = nh + (v_is_k ? 1 : 2) * nkv;
   int lanes_per_head = 1;
   while (lanes_per_head * 16 < hd) lanes_per_head *= 2;
   const int heads_per_warp = 32 / lanes_per_head;
@@ -323,13 +339,13 @@ extern "C" int hb_qkv_post(const void* qkv, int dtype, const float* inv_freq, in
   if (dtype == HB_DTYPE_F32)
     qkv_post_kernel<float><<<grid, threads, 0, stream>>>(
         (const float*)qkv, inv_freq, rot_pairs, interleaved, qk_norm, qk_eps, temp_on, floor_scale, attn_scale,
-        q_norm_w, k_norm_w, norm_first, rot_mul,
+        q_norm_w, k_norm_w, norm_first, rot_mul, v_is_k,
         positions, seq_of_token, block_table, table_stride, (float*)q_out, (float*)k_pages, (float*)v_pages,
         page_size, write_kv, n_tokens, nh, nkv, hd, lanes_per_head);
   else if (dtype == HB_DTYPE_BF16)
     qkv_post_kernel<__nv_bfloat16><<<grid, threads, 0, stream>>>(
         (const __nv_bfloat16*)qkv, inv_freq, rot_pairs, interleaved, qk_norm, qk_eps, temp_on, floor_scale,
-        attn_scale, q_norm_w, k_norm_w, norm_first, rot_mul, positions, seq_of_token, block_table, table_stride,
+        attn_scale, q_norm_w, k_norm_w, norm_first, rot_mul, v_is_k, positions, seq_of_token, block_table, table_stride,
         (__nv_bfloat16*)q_out,
         (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, page_size, write_kv, n_tokens, nh, nkv, hd, lanes_per_head);
   else

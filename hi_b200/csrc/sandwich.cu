@@ -2,7 +2,7 @@
 //
 //   y = delta + delta2 + sum_j routed[slot_j] * weight_j       the sub-layer's open result (any part absent)
 //   x <- x + y rsqrt(mean(y^2) + eps_y) w_y                     the stream, float32, in place
-//   h = x rsqrt(mean(x^2) + eps) w                              the next sub-layer's input (w null: not wanted)
+//   h = x rsqrt(mean(x^2) + eps) w                              the next sub-layer's input (w null: h = x, where y is given)
 //
 // One kernel a boundary: the stream is read and written once. With `row_map` only those rows are taken and the stream
 // is left as it is (the rows whose logits are wanted). Norm weights are float32 as they act (a weight stored around
@@ -78,6 +78,10 @@ __global__ void sandwich_kernel(const SandwichArgs a) {
     if (!a.row_map) a.x[src * a.hidden + j] = s;
     row_s[j] = s;
     ss += s * s;
+    if (!a.w && a.y) {
+      if (a.y_dtype == HB_DTYPE_F32) reinterpret_cast<float*>(a.y)[src * a.hidden + j] = s;
+      else reinterpret_cast<__nv_bfloat16*>(a.y)[src * a.hidden + j] = __float2bfloat16_rn(s);
+    }
   }
   if (!a.w) return;
   const float inv = rsqrtf(hb::block_sum(ss, scratch) / (float)a.hidden + a.eps);
@@ -138,6 +142,7 @@ __global__ void __launch_bounds__(512) sandwich_vec_kernel(const SandwichArgs a)
       s = make_float4(xv[g].x + s.x * inv_y * wy[g].x, xv[g].y + s.y * inv_y * wy[g].y, xv[g].z + s.z * inv_y * wy[g].z,
                       xv[g].w + s.w * inv_y * wy[g].w);
       if (!a.row_map) *reinterpret_cast<float4*>(a.x + src * a.hidden + idx) = s;
+      if (!a.w && a.y) st4(a.y, a.y_dtype, src * a.hidden + idx, s);
       v[g] = s;
       ss += dot4(s);
     }
@@ -164,7 +169,7 @@ extern "C" int hb_sandwich_step(float* x, const void* delta, int delta_dtype, co
                                 const float* w_y, float eps_y, const float* w, float eps, void* y, int y_dtype, float* y_f32,
                                 const int* row_map, int rows, int hidden, cudaStream_t stream) {
   if (!x || !w_y || rows < 0 || hidden <= 0 || (delta && !known(delta_dtype)) || (delta2 && !known(delta2_dtype)) ||
-      (w && (!y || !known(y_dtype))) || (!w && row_map))
+      (w && !y) || (y && !known(y_dtype)) || (!w && row_map))
     return HB_ERR_BAD_ARG;
   if (routed && (!slot_of_entry || top_k < 1 || top_k > 8)) return HB_ERR_BAD_ARG;
   if (rows == 0) return HB_OK;

@@ -34,12 +34,12 @@ _SIGNATURES = {
     "hb_softcap": [P, F, c_longlong, P],
     "hb_convert": [P, I, P, I, c_longlong, P],
     "hb_moe_combine": [P, P, P, P, I, P, I, I, I, P],
-    "hb_qkv_post": [P, I, P, I, I, I, F, I, F, F, P, P, I, I, F, P, I, I, P, P, P, I, P, P, P, I, I, I, I, I, I, P],
+    "hb_qkv_post": [P, I, P, I, I, I, F, I, F, F, P, P, I, I, F, P, I, I, I, P, P, P, I, P, P, P, I, I, I, I, I, I, P],
     "hb_paged_attention": [P, I, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, F, P, P, I, I, P, P, P],
     "hb_attention_merge": [P, P, P, I, I, I, I, I, I, P, P],
     "hb_attention_decode": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, P, F, P, P, I, I, P, P, P],
     "hb_attention_decode_tma": [P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, F, I, I, I, P, P, P, P],
-    "hb_attention_decode_fused": [P, P, I, I, I, F, I, F, F, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, F, I, I, P, P, P, P, P, P, I, F, I, P],
+    "hb_attention_decode_fused": [P, P, I, I, I, F, I, F, F, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, F, I, I, P, P, P, P, P, P, I, F, I, I, P],
     "hb_attention_prefill": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P],
     "hb_attention_prefill_reshaped": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, F, I, I, F, P, P, P, P, P],
     "hb_attention_prefill_tc": [P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, I, P, I, P, P, P, P],
@@ -894,7 +894,8 @@ def qkv_post(qkv: torch.Tensor, nh: int, nkv: int, hd: int, positions: torch.Ten
              v_pages: Optional[torch.Tensor], page_size: int, write_kv: bool,
              q_norm_weight: Optional[torch.Tensor] = None, k_norm_weight: Optional[torch.Tensor] = None,
              norm_first: bool = False, norm_dim: int = 0, rot_mul: float = 1.0,
-             v_inv_freq: Optional[torch.Tensor] = None, v_interleaved: bool = False) -> torch.Tensor:
+             v_inv_freq: Optional[torch.Tensor] = None, v_interleaved: bool = False,
+             values_are_keys: bool = False) -> torch.Tensor:
     """Rotary or temperature, optional L2 norm, and the cache append; returns q [N, nh, hd].
 
     By default the norm of q and k is weightless and comes after the rotation. ``norm_first``: it comes
@@ -903,16 +904,20 @@ def qkv_post(qkv: torch.Tensor, nh: int, nkv: int, hd: int, positions: torch.Ten
     cos and sin. Any even number of rotating dims is taken then (a general kernel runs these forms).
     ``v_inv_freq`` (float32 [pairs]): the values are cached rotated by their own position, pair m of their first
     2 * pairs dims by position * v_inv_freq[m] (pairs (m, m + pairs), or (2m, 2m + 1) with ``v_interleaved``).
+    ``values_are_keys``: ``qkv`` is [N, (nh + nkv) * hd] and a key head as projected, before norm and rotation, is also
+    the value.
 
     ``qkv`` is [N, (nh + 2*nkv) * hd]; ``k_pages``/``v_pages`` are [pages, nkv, page_size, hd];
     ``block_table`` [S, width] int32 maps (sequence row, position // page_size) to a page.
     """
     _need(qkv, "qkv"); _need(positions, "positions", torch.int32)
-    n = qkv.shape[0]
-    if qkv.shape[1] != (nh + 2 * nkv) * hd:
-        raise KernelError(f"qkv has {qkv.shape[1]} columns, expected {(nh + 2 * nkv) * hd}")
+    n, columns = qkv.shape[0], (nh + (1 if values_are_keys else 2) * nkv) * hd
+    if qkv.shape[1] != columns:
+        raise KernelError(f"qkv has {qkv.shape[1]} columns, expected {columns}")
+    if values_are_keys and v_inv_freq is not None:
+        raise KernelError("values that are the projected keys are not rotated")
     general = v_inv_freq is not None or norm_first or q_norm_weight is not None or k_norm_weight is not None or rot_mul != 1.0 or \
-        (norm_dim not in (0, hd)) or (inv_freq is not None and inv_freq.numel() % 8 != 0)
+        (norm_dim not in (0, hd)) or (inv_freq is not None and inv_freq.numel() % 8 != 0) or (values_are_keys and hd > 256)
     if hd % 8 != 0 or hd > 1024 or (not general and (hd % 16 != 0 or hd > 256)):
         raise KernelError(f"head_dim {hd} is not supported (multiples of 16 up to 256; the general form: of 8 up to 1024)")
     v_pairs = 0
@@ -945,7 +950,7 @@ def qkv_post(qkv: torch.Tensor, nh: int, nkv: int, hd: int, positions: torch.Ten
     _check(lib().hb_qkv_post(_ptr(qkv), _dt(qkv), _ptr(inv_freq), rot_pairs, int(interleaved), int(qk_norm),
                              float(qk_eps), int(temperature is not None), float(fs), float(asc), _ptr(q_norm_weight),
                              _ptr(k_norm_weight), int(norm_first), int(norm_dim), float(rot_mul), _ptr(v_inv_freq),
-                             v_pairs, int(v_interleaved), _ptr(positions),
+                             v_pairs, int(v_interleaved), int(values_are_keys), _ptr(positions),
                              _ptr(seq_of_token), _ptr(block_table), stride, _ptr(q), _ptr(k_pages), _ptr(v_pages),
                              page_size, int(write_kv), n, nh, nkv, hd, _stream()), "qkv_post")
     return q
@@ -1275,20 +1280,21 @@ def decode_attention_fused(qkv: torch.Tensor, nh: int, nkv: int, hd: int, positi
                            block_table: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, chunk: int,
                            window: int, scale: float, max_context: int, merge_inside: bool = True,
                            q_norm_weight: Optional[torch.Tensor] = None, k_norm_weight: Optional[torch.Tensor] = None,
-                           norm_first: bool = False, rot_mul: float = 1.0, sink: bool = False) -> Optional[torch.Tensor]:
+                           norm_first: bool = False, rot_mul: float = 1.0, sink: bool = False,
+                           values_are_keys: bool = False) -> Optional[torch.Tensor]:
     """:func:`qkv_post`, :func:`decode_attention` and the merge of its splits in ONE launch, for a step
     of single decoded tokens: ``qkv`` [N, (nh + 2 nkv) * hd] bfloat16 is the projection's output; the
     kernel encodes q, k and v, appends the token's key and value to its page, attends over the cache
     and combines the splits (the block that finishes last does it). Returns [N, nh, hd], or None
     where the kernel does not take the shapes (the caller then runs the three kernels). ``q_norm_weight``,
-    ``k_norm_weight``, ``norm_first``, ``rot_mul`` and ``sink`` as in :func:`qkv_post` and :func:`paged_attention`
+    ``k_norm_weight``, ``norm_first``, ``rot_mul``, ``values_are_keys`` and ``sink`` as in :func:`qkv_post` and :func:`paged_attention`
     (the norm then runs over the whole head)."""
     _need(qkv, "qkv", torch.bfloat16); _need(k_pages, "k_pages", qkv.dtype); _need(v_pages, "v_pages", qkv.dtype)
     for t, nm in ((block_table, "block_table"), (seq_of_token, "seq_of_token"), (positions, "positions")):
         _need(t, nm, torch.int32)
     n = qkv.shape[0]
     n_pages, nkv2, page_size, hd2 = k_pages.shape
-    if qkv.shape[1] != (nh + 2 * nkv) * hd or hd2 != hd or nkv2 != nkv or k_pages.shape != v_pages.shape:
+    if qkv.shape[1] != (nh + (1 if values_are_keys else 2) * nkv) * hd or hd2 != hd or nkv2 != nkv or k_pages.shape != v_pages.shape:
         raise KernelError("qkv or the cache pages do not match the heads and head_dim")
     if not decode_attention_supported(qkv.dtype, nh, nkv, hd) or n * nkv > min(FUSED_COUNTERS, FUSED_MAX_GROUPS):
         return None
@@ -1318,7 +1324,7 @@ def decode_attention_fused(qkv: torch.Tensor, nh: int, nkv: int, hd: int, positi
         _ptr(positions), _ptr(out), n, nh, nkv, hd, page_size, int(chunk), int(window), float(scale), split_size, splits,
         _ptr(part_acc), _ptr(part_ml), _ptr(_fused_counter_buffer(qkv.device)) if merge_inside else None,
         _ptr(_tc_status(qkv.device)), _ptr(q_norm_weight), _ptr(k_norm_weight), int(norm_first), float(rot_mul), int(sink),
-        _stream())
+        int(values_are_keys), _stream())
     if code == _UNSUPPORTED:
         return None
     TC_USED[0] = True
@@ -1571,7 +1577,8 @@ def sandwich_step(x: torch.Tensor, y_weight: torch.Tensor, y_eps: float, delta: 
                   routed_weight: Optional[torch.Tensor] = None, weight: Optional[torch.Tensor] = None, eps: float = 0.0,
                   out_dtype: Optional[torch.dtype] = None, row_map: Optional[torch.Tensor] = None, also_f32: bool = False):
     """``x += rmsnorm(delta + delta2 + routed rows) * y_weight`` (float32, in place), then, with ``weight``,
-    ``rmsnorm(x) * weight`` in ``out_dtype`` (returned; None without ``weight``). ``routed``, ``slot_of_entry``,
+    ``rmsnorm(x) * weight`` in ``out_dtype`` (returned). Without ``weight``: x itself in ``out_dtype``, where that is
+    given, else None. ``routed``, ``slot_of_entry``,
     ``routed_weight``, ``row_map`` and ``also_f32`` as :func:`add_rmsnorm`; the weights are float32."""
     _need(x, "x", torch.float32); _need(y_weight, "y_weight", torch.float32)
     rows_total, hidden = x.shape
@@ -1596,10 +1603,10 @@ def sandwich_step(x: torch.Tensor, y_weight: torch.Tensor, y_eps: float, delta: 
         if routed_weight is not None:
             _need(routed_weight, "routed_weight", torch.float32)
     y = y32 = None
-    if weight is not None:
+    if weight is not None or out_dtype is not None:
         y = torch.empty((rows, hidden), dtype=out_dtype, device=x.device)
-        if also_f32 and out_dtype != torch.float32:
-            y32 = torch.empty((rows, hidden), dtype=torch.float32, device=x.device)
+    if weight is not None and also_f32 and out_dtype != torch.float32:
+        y32 = torch.empty((rows, hidden), dtype=torch.float32, device=x.device)
     _check(lib().hb_sandwich_step(_ptr(x), _ptr(delta), _dt(delta) if delta is not None else 0, _ptr(delta2),
                                   _dt(delta2) if delta2 is not None else 0, _ptr(routed), _ptr(slot_of_entry),
                                   _ptr(routed_weight) if routed is not None else None, int(top_k), _ptr(y_weight),

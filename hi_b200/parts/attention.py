@@ -205,9 +205,11 @@ class AttentionMixer(Part):
                        o = a1 - lambda a2 with lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + c (one number a layer,
                        ``<prefix>.lq1|lk1|lq2|lk2`` [head_dim]), and o <- o / rms(o) (over the head's values, eps
                        ``qk_norm_eps``) * (1 - c)
+      ``values``       "projected" (default) | "keys": there is no value projection; a key as projected, before norm and
+                       rotation, is its value too (``value_dim`` is then ``head_dim``)
       ``output_gate``  the heads' results are multiplied element by element by sigmoid(W_g h), ``<prefix>.g``
                        [heads * value_dim, H], before the output projection
-    tensors: the four projections, and each projection's bias where the checkpoint has one (a bias is
+    tensors: the four projections (without ``v`` where the values are the keys), and each projection's bias where the checkpoint has one (a bias is
     used iff its tensor exists: crates/hi-mlx/src/models.rs:1808, 1843-1845).
     """
 
@@ -241,6 +243,12 @@ class AttentionMixer(Part):
         self.diff = float(p["differential"]) if p.get("differential") is not None else None
         self.gated = bool(p.get("output_gate", False))
         self.maps = 1 if self.diff is None else 2
+        self.values_are_keys = p.get("values", "projected") == "keys"
+        if p.get("values", "projected") not in ("projected", "keys"):
+            raise ValueError(f"{prefix}: values are 'projected' or 'keys'")
+        if self.values_are_keys and (self.vdim != self.dim or self.sigmoid or self.taps or self.diff is not None or p.get("output_gate")):
+            raise ValueError(f"{prefix}: values that are the keys are built for softmax weights, one head size, no convolution, "
+                             f"second map or output gate")
         # these work on the unpadded projection (ops.conv_qkv encodes and appends)
         self.unpadded = bool(self.taps) or self.diff is not None or self.gated
         if self.unpadded and (self.sigmoid or p.get("temperature") or (p.get("qk_norm") and not self.norm_weighted)):
@@ -258,7 +266,7 @@ class AttentionMixer(Part):
                 self.hd = next((r for r in ops.TC_ROW_LENGTHS if r >= self.hd), self.hd)
         elif self.dim != self.vdim or self.dim % 16:
             self.hd = -(-max(self.dim, self.vdim) // 16) * 16                  # rows of the cache and of q
-        if self.hd > (1024 if self.hd != self.dim or self.norm_weighted or self.unpadded else 256):
+        if self.hd > (1024 if self.hd != self.dim or self.norm_weighted or self.unpadded or self.values_are_keys else 256):
             raise ValueError(f"{prefix}: head size {self.hd} is not supported")
         self.window = tuple(p["window"]) if p.get("window") else None
         self.keep = int(self.window[2]) if self.window and len(self.window) > 2 else 0
@@ -292,10 +300,11 @@ class AttentionMixer(Part):
         h, nh, nkv = self.hidden, self.nh, self.nkv
         have = "qkvo" if self.bias is True else (self.bias or "")
         rows = {"q": nh * self.maps * self.dim, "k": nkv * self.maps * self.dim, "v": nkv * self.vdim, "o": h}
-        specs = [TensorSpec(self._name(n), (rows[n], h) if n != "o" else (h, nh * self.vdim)) for n in "qkvo"]
+        names = "qko" if self.values_are_keys else "qkvo"
+        specs = [TensorSpec(self._name(n), (rows[n], h) if n != "o" else (h, nh * self.vdim)) for n in names]
         # "absent": the random-weights writer leaves them out
         specs += [TensorSpec(self._name(n, bias=True), (rows[n],), init="normal" if n in have else "absent", optional=True)
-                  for n in "qkvo"]
+                  for n in names]
         if self.norm_weighted:
             specs += [TensorSpec(f"{self.prefix}.{n}.norm", (self.dim,), init="ones") for n in "qk"]
         if self.sigmoid:
@@ -365,17 +374,17 @@ class AttentionMixer(Part):
     def load(self, fetch):
         if self.unpadded:
             return self._load_unpadded(fetch)
-        q, k, v = (fetch(self._name(n)) for n in "qkv")
-        if not (q.dtype == k.dtype == v.dtype):
-            q, k, v = q.float(), k.float(), v.float()
-        sizes = ((self.nh, self.dim), (self.nkv, self.dim), (self.nkv, self.vdim))
-        q, k, v = (self._pad_heads(t, *hs) for t, hs in zip((q, k, v), sizes))
-        self.w_qkv = torch.cat([q, k, v], dim=0).contiguous()     # one product for q, k and v
+        names = "qk" if self.values_are_keys else "qkv"
+        rows = [fetch(self._name(n)) for n in names]
+        if len({t.dtype for t in rows}) > 1:
+            rows = [t.float() for t in rows]
+        sizes = ((self.nh, self.dim), (self.nkv, self.dim), (self.nkv, self.vdim))[: len(names)]
+        self.w_qkv = torch.cat([self._pad_heads(t, *hs) for t, hs in zip(rows, sizes)], dim=0).contiguous()     # one product
         w_o = fetch(self._name("o"))
         if self.vdim != self.hd:
             w_o = self._pad_heads(w_o.t().contiguous(), self.nh, self.vdim).t()
         self.w_o = w_o.contiguous()
-        biases = [fetch(self._name(n, bias=True)) for n in "qkv"]
+        biases = [fetch(self._name(n, bias=True)) for n in names]
         if any(b is not None for b in biases):          # a projection without one adds zeros
             biases = [torch.zeros(hs[0] * self.hd, dtype=self.w_qkv.dtype, device=self.w_qkv.device) if b is None
                       else self._pad_heads(b, *hs) for b, hs in zip(biases, sizes)]
@@ -432,6 +441,8 @@ class AttentionMixer(Part):
         table = self.position.rotary_table()
         if table is None and hasattr(self.position, "apply"):
             # a position part without a rotary table encodes q and k itself
+            if self.values_are_keys:
+                raise TypeError(f"{self.prefix}: values that are the keys need a position part with a rotary table")
             n = qkv.shape[0]
             q, k, v = qkv.split([self.nh * self.hd, self.nkv * self.hd, self.nkv * self.hd], dim=1)
             q, k = self.position.apply(q.reshape(n, self.nh, self.hd), k.reshape(n, self.nkv, self.hd), positions)
@@ -462,14 +473,15 @@ class AttentionMixer(Part):
                                            self.qk_norm_eps, self.temperature, ctx.seq_of_token, block_table,
                                            cache.k_pages, cache.v_pages, chunk, sliding, self.scale, ctx.max_context,
                                            q_norm_weight=self.w_qnorm, k_norm_weight=self.w_knorm,
-                                           norm_first=self.norm_weighted, rot_mul=rot_mul, sink=self.sink)
+                                           norm_first=self.norm_weighted, rot_mul=rot_mul, sink=self.sink,
+                                           values_are_keys=self.values_are_keys)
             if o is not None:
                 return linear(o.view(o.shape[0], self.nh * self.hd), self.w_o, bias=self.b_o)
         q = ops.qkv_post(qkv, self.nh, self.nkv, self.hd, positions, inv_freq, interleaved, self.qk_norm,
                          self.qk_norm_eps, self.temperature, ctx.seq_of_token, block_table, cache.k_pages,
                          cache.v_pages, ctx.page_size, cache.writes, q_norm_weight=self.w_qnorm,
                          k_norm_weight=self.w_knorm, norm_first=self.norm_weighted,
-                         norm_dim=0 if plain else self.dim, rot_mul=rot_mul)
+                         norm_dim=0 if plain else self.dim, rot_mul=rot_mul, values_are_keys=self.values_are_keys)
         o = attend_over_pages(q, cache.k_pages, cache.v_pages, block_table, ctx, self.nh, self.nkv, self.hd, chunk,
                               sliding, self.scale, sink=self.sink, softcap=self.softcap, slopes=self.slopes,
                               sink_values=self.sink_values, keep=self.keep)

@@ -186,8 +186,11 @@ def llama3_inverse_frequencies(head_dim: int, theta: float, scaling: Optional[di
 
 def exact_inverse_frequencies(dims: int, theta: float, scaling: Optional[dict]) -> np.ndarray:
     """The table of :func:`llama3_inverse_frequencies` (same keys of ``scaling``) worked out in float64 and
-    rounded to float32 once."""
+    rounded to float32 once. ``scaling`` = {"factor"} alone: every frequency is divided by it."""
     out = np.empty(dims // 2, dtype=np.float64)
+    if scaling and set(scaling) == {"factor"}:
+        out[:] = [float(theta) ** (-2.0 * j / dims) / float(scaling["factor"]) for j in range(dims // 2)]
+        return out.astype(np.float32)
     for j in range(dims // 2):
         inv = float(theta) ** (-2.0 * j / dims)
         if scaling:
@@ -483,6 +486,54 @@ class SandwichBlock(Part):
                 h = layer.norm_feed_forward.forward(residual, pending)
                 y = layer.feed_forward.forward(h, ctx)
             pending = self._open(1, y)
+        return residual, pending
+
+
+@register("arrangement", "normed_output")
+class NormedOutputBlock(Part):
+    """A norm on what a sub-layer returns and none on what it reads: x <- x + mult * norm1(mixer(x));
+    x <- x + mult * norm2(ff(x)).
+
+    The residual stream is float32; the sub-layers read its rounding to the engine's dtype, routers the stream itself. A
+    sub-layer's result stays open (:class:`~hi_b200.parts.context.NormedPending`): the next boundary, one kernel, takes it
+    through its norm, sums it into the stream and writes the rounding beside it; behind the last layer the model's norm
+    does so. A layer without feed-forward has the first half only.
+
+    params: ``mult`` (default 1). The norms of the layer must be ``rmsnorm``."""
+
+    graph_safe = True
+
+    def __init__(self, params, prefix, env):
+        super().__init__(params, prefix, env)
+        self.mult = float(params.get("mult", 1.0))
+        self._weights: Dict[int, torch.Tensor] = {}
+
+    def _open(self, norm, delta):
+        # the factor rides on the norm's weight (float32), worked out once
+        if id(norm) not in self._weights:
+            self._weights[id(norm)] = norm.weight_f32 * self.mult if self.mult != 1.0 else norm.weight_f32
+        return NormedPending(delta=delta, weight=self._weights[id(norm)], eps=norm.eps)
+
+    def forward(self, layer, residual, pending, ctx, cache_view):
+        norm1, norm2 = layer.norm_mixer, layer.norm_feed_forward
+        if not isinstance(norm1, RMSNorm) or (norm2 is not None and not isinstance(norm2, RMSNorm)):
+            raise TypeError(f"{self.prefix}: the block works with rmsnorm norms")
+        if pending is None:
+            h = residual if residual.dtype == self.env.dtype else ops.convert(residual, self.env.dtype)
+        elif isinstance(pending, NormedPending):
+            h = pending.read(residual, self.env.dtype)
+        else:
+            raise TypeError(f"{self.prefix}: the block before this one left a sum open that no norm takes")
+        if ctx.tap is not None:
+            ctx.tap(f"{self.prefix}.stream_in", residual)        # debug: the stream as this layer reads it
+        pending = self._open(norm1, layer.mixer.forward(h, ctx, cache_view))
+        if layer.feed_forward is not None:
+            h = pending.read(residual, self.env.dtype)
+            if getattr(layer.feed_forward, "wants_f32_input", False):
+                y = layer.feed_forward.forward(h, ctx, normed_f32=residual)
+            else:
+                y = layer.feed_forward.forward(h, ctx)
+            pending = self._open(norm2, y)
         return residual, pending
 
 

@@ -132,6 +132,15 @@ class NormedPending:
 
         ops.sandwich_step(residual, self.weight, self.eps, **self.parts(residual.shape[0]))
 
+    def read(self, residual: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+        """Into the stream, for a consumer that reads the stream itself: its rounding to ``dtype``, written by the same
+        kernel (the stream, where that has the dtype already)."""
+        from ..kernels import ops
+
+        y = ops.sandwich_step(residual, self.weight, self.eps, out_dtype=None if dtype == residual.dtype else dtype,
+                              **self.parts(residual.shape[0]))
+        return residual if y is None else y
+
 
 @dataclass
 class HyperPending:

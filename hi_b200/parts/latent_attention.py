@@ -40,8 +40,10 @@ class LatentAttentionMixer(Part):
     params: ``hidden_size``, ``heads``, ``dim``, ``vdim``, ``kv_rank``, ``scale``, ``eps`` (of the latents'
     norms), ``own_latents`` (False for a layer that reads another's), ``window`` (None | ("sliding", W) |
     ("chunk", C): which earlier latents a query reads; default all), ``gate`` (default True: the sigmoid gate
-    per head), ``q_rank`` (default None: queries straight from h), ``rot_dim`` (default 0), ``rot_base``,
-    ``rot_scaling`` (None | the keys of :func:`~hi_b200.parts.basic.exact_inverse_frequencies`),
+    per head; "element": W_g has a row per value element, o *= sigmoid(W_g h) element by element), ``sink`` (default
+    False; True: the softmax's denominator has one more term exp(sink_a), a learned number per head that is not scaled
+    and has no value), ``q_rank`` (default None: queries straight from h), ``rot_dim`` (default 0), ``rot_base``,
+    ``rot_scaling`` (None | {"factor"}: every frequency is divided by it | the keys of :func:`~hi_b200.parts.basic.exact_inverse_frequencies`),
     ``rot_kind`` ("llama3", the default | "yarn": ``rot_scaling`` = {factor, original, fast, slow}, the ramped
     frequencies of :func:`~hi_b200.parts.basic.yarn_inverse_frequencies` and their factor on cos and sin, which
     both the query's and the key's rotated part carry), ``rot_interleaved`` (pairs (2i, 2i + 1) instead of
@@ -49,7 +51,8 @@ class LatentAttentionMixer(Part):
     tensors: ``<prefix>.q`` [heads*dim, H] (or ``<prefix>.dq`` [q_rank, H], ``<prefix>.dq.norm`` [q_rank],
     ``<prefix>.uq`` [heads*(dim+rot_dim), q_rank]), ``<prefix>.dkv`` [rank+rot_dim, H] and ``<prefix>.dkv.norm``
     [rank] (own latents only), ``<prefix>.uk`` [heads*dim, rank], ``<prefix>.uv`` [heads*vdim, rank],
-    ``<prefix>.g`` [heads, H] (with ``gate``), ``<prefix>.o`` [H, heads*vdim].
+    ``<prefix>.g`` [heads, H] (with ``gate``; "element": [heads*vdim, H]), ``<prefix>.sink`` [heads] (with ``sink``),
+    ``<prefix>.o`` [H, heads*vdim].
     """
 
     graph_safe = True
@@ -64,6 +67,9 @@ class LatentAttentionMixer(Part):
         self.own = bool(p.get("own_latents", True))
         self.window = tuple(p["window"]) if p.get("window") else None
         self.gate = bool(p.get("gate", True))
+        self.gate_elements = p.get("gate", True) == "element"
+        self.sink = bool(p.get("sink", False))
+        self.sink_values: Optional[torch.Tensor] = None
         self.q_rank = int(p["q_rank"]) if p.get("q_rank") else 0
         self.rot = int(p.get("rot_dim") or 0)
         if self.rot % 2:
@@ -100,7 +106,9 @@ class LatentAttentionMixer(Part):
             specs += [TensorSpec(f"{pre}.dkv", (r + self.rot, h)), TensorSpec(f"{pre}.dkv.norm", (r,), init="ones")]
         specs += [TensorSpec(f"{pre}.uk", (hd, r)), TensorSpec(f"{pre}.uv", (hv, r))]
         if self.gate:
-            specs.append(TensorSpec(f"{pre}.g", (self.heads, h)))
+            specs.append(TensorSpec(f"{pre}.g", (hv if self.gate_elements else self.heads, h)))
+        if self.sink:
+            specs.append(TensorSpec(f"{pre}.sink", (self.heads,)))
         return specs + [TensorSpec(f"{pre}.o", (h, hv))]
 
     def load(self, fetch):
@@ -108,10 +116,20 @@ class LatentAttentionMixer(Part):
         q = fetch(f"{pre}.dq" if self.q_rank else f"{pre}.q")
         parts = [q]
         self.n_q = q.shape[0]
+
+        def align():                     # zero rows: the next columns of the product start on 16 bytes
+            short = -sum(t.shape[0] for t in parts) % 8
+            if self.gate_elements and short:
+                parts.append(torch.zeros((short, self.hidden), dtype=q.dtype, device=q.device))
+            return sum(t.shape[0] for t in parts)
+
+        self.off_g = self.off_kv = align()
         if self.gate:
             parts.append(fetch(f"{pre}.g"))
+            self.off_kv = align()
         if self.own:
             parts.append(fetch(f"{pre}.dkv"))
+            align()
             self.w_c = fetch(f"{pre}.dkv.norm").to(q.dtype).contiguous()
         # one product for the queries (or their latent), the gates and (own latents) the down projection
         self.w_in = torch.cat([t.to(q.dtype) for t in parts], dim=0).contiguous()
@@ -127,6 +145,8 @@ class LatentAttentionMixer(Part):
         self.w_uk = uk.contiguous()                              # [heads, dim, row_len]: q_a -> latent space
         self.w_uv_t = uv.transpose(1, 2).contiguous()            # [heads, row_len, vdim]: latent space -> o_a
         self.w_o = fetch(f"{pre}.o").contiguous()
+        if self.sink:
+            self.sink_values = fetch(f"{pre}.sink").to(torch.float32).contiguous()
         if self.rot:
             self._freq = torch.from_numpy(self._freq_host).to(self.w_in.device)
 
@@ -136,10 +156,8 @@ class LatentAttentionMixer(Part):
         block_table = ctx.block_tables[cache.group]
         if self.own != cache.writes:
             raise RuntimeError(f"{self.prefix}: a layer with its own latents writes its cache slot, another reads one")
-        off_g = self.n_q
-        off_kv = off_g + (self.heads if self.gate else 0)
         if self.own:
-            ops.latent_append(proj[:, off_kv:], self.w_c, self.eps, ctx.positions, ctx.seq_of_token, block_table,
+            ops.latent_append(proj[:, self.off_kv: self.off_kv + self.rank + self.rot], self.w_c, self.eps, ctx.positions, ctx.seq_of_token, block_table,
                               cache.k_pages, inv_freq=self._freq, interleaved=self.rot_interleaved, rot_mul=self.rot_mul)
         if self.q_rank:
             q = linear(ops.rmsnorm_rows(proj[:, : self.q_rank], self.w_qn, self.eps), self.w_uq)
@@ -156,9 +174,11 @@ class LatentAttentionMixer(Part):
         chunk = self.window[1] if self.window and self.window[0] == "chunk" else 0
         sliding = self.window[1] if self.window and self.window[0] == "sliding" else 0
         o_lat = attend_over_pages(q_lat, cache.k_pages, cache.k_pages, block_table, ctx, self.heads, 1, self.row_len,
-                                  chunk, sliding, self.scale)
+                                  chunk, sliding, self.scale, sink_values=self.sink_values)
         o = torch.empty((n, self.heads, self.vdim), dtype=proj.dtype, device=proj.device)
         torch.bmm(o_lat.transpose(0, 1), self.w_uv_t, out=o.transpose(0, 1))
-        if self.gate:
-            o = ops.head_gate(o, proj[:, off_g: off_g + self.heads])
+        if self.gate_elements:
+            o = ops.gate_rows(o, proj[:, self.off_g: self.off_g + self.heads * self.vdim], self.vdim)
+        elif self.gate:
+            o = ops.head_gate(o, proj[:, self.off_g: self.off_g + self.heads])
         return linear(o.view(n, self.heads * self.vdim), self.w_o)
