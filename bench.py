@@ -1617,6 +1617,197 @@ def case_fofisun_step(tokens=2048, batch=8, context=4096, width=2048, heads=16, 
     torch.cuda.synchronize()
 
 
+# --------------------------------------------------------------------------- Darotar beside the closest existing models
+def _darotar_config(width, heads, ff, layers, vocab=32000, window=4096):
+    """Layers in the order latent attention (heads of 128 + 64 rotated over a latent of 128), windowed attention (heads of
+    128, a quarter as many key heads, which are the values too), latent attention that reads the first one's latents; 8
+    experts of half the dense size, 2 a token."""
+    moe = {"kind": "moe", "expert": {"ff": ff // 2}, "router": {"experts": 8, "top": 2}}
+
+    def latent(source=None):
+        m = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 128, "q_rank": width // 2, "scale": 192 ** -0.5,
+             "rot": {"base": 500000.0, "dims": 64}}
+        return {"type": "latent_attention", "mlp": moe, "mixer": m if source is None else {**m, "kv_from": source}}
+    att = {"type": "attention", "mlp": moe, "mixer": {
+        "heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window},
+        "rot": {"base": 10000.0, "dims": 128, "scaling": {"factor": 8.0}}}}
+    order = [(latent(), att, latent(i - 2))[i % 3] for i in range(layers)]
+    return {"architecture": "Darotar", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.4, "layers": order}
+
+
+def case_darotar(width=2048, heads=16, ff=8192, layers=6, tokens=2048, batch=8, context=4096):
+    """Prefill (one prompt of ``tokens`` in one step) and decode (``batch`` requests at ``context`` cached tokens,
+    captured steps) throughput of a Darotar model with random weights beside Bezasun (the closest existing model:
+    latent attention, attention and routed experts) and a dense Llama-4-shaped model of equal width, depth and heads; then
+    the extended kernels alone beside their like kernels, with the bytes that must move over the measured copy bandwidth.
+    Markdown on standard output."""
+    import torch
+
+    from hi_b200.engine.core import Engine, StepEntry
+    from hi_b200.kernels import ops
+
+    pk = peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=DEV)
+    g = torch.Generator().manual_seed(0)
+
+    def timed(fn, reps=9, flush_l2=True):
+        for _ in range(3):
+            fn()
+        ts = []
+        for _ in range(reps):
+            if flush_l2:
+                flush.zero_()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record(); fn(); b.record()
+            torch.cuda.synchronize()
+            ts.append(a.elapsed_time(b))
+        return sorted(ts)[len(ts) // 2]
+
+    print(f"peaks: {pk['hbm_gbs']:.0f} GB/s copy, {pk['bf16_tflops']:.0f} TFLOP/s bf16 ({pk['source']}); "
+          f"width {width}, {heads} heads, feed-forward {ff}, {layers} layers, bf16, random weights\n")
+    print("| model | prefill tokens/s | ms | decode tokens/s | ms/step | weights GB | launches/decode step |\n|---|---|---|---|---|---|---|")
+    for name, cfg in (("Darotar", _darotar_config(width, heads, ff, layers)), ("Bezasun", _bezasun_config(width, heads, ff, layers)),
+                      ("dense Llama-4 shape", _dense_llama_config(width, heads, ff, layers))):
+        eng = Engine.from_config(cfg, seed=0, dtype="bfloat16", device=DEV, kv_page_size=PAGE,
+                                 kv_cache_tokens=batch * (context + 256) + tokens + 256, max_active_requests=batch + 1)
+        vocab = eng.vocab_size
+        weights = sum(2 * int(torch.Size(sp.shape).numel()) for sp in eng.model.tensor_specs() if sp.init != "absent") / 1e9
+        prompt = torch.randint(0, vocab, (tokens,), generator=g).tolist()
+
+        def prefill():
+            eng.step([StepEntry("p", prompt, [tokens - 1])])
+            eng.finish("p")
+        t_pre = timed(prefill, reps=5)
+        for i in range(batch):
+            eng.assume_cached(i, context)
+        toks = torch.randint(0, vocab, (64, batch), generator=g).tolist()
+        turn = [0]
+
+        def decode():
+            eng.step([StepEntry(i, [toks[turn[0] % 64][i]], [0]) for i in range(batch)], borrow=True)
+            turn[0] += 1
+        for _ in range(4):
+            decode()
+        before = ops.LAUNCHES[0]
+        t_dec = timed(decode, reps=9, flush_l2=False)
+        launches = (ops.LAUNCHES[0] - before) // 12
+        print(f"| {name} | {tokens / t_pre * 1e3:,.0f} | {t_pre:.2f} | {batch / t_dec * 1e3:,.0f} | {t_dec:.3f} | {weights:.2f} | {launches} |")
+        del eng
+        torch.cuda.empty_cache()
+    rows = _darotar_kernels(width, heads, ff, tokens, batch, context, timed, pk)
+    print("\n| step | kernel | us | MB that must move | GB/s | of the copy peak | |\n|---|---|---|---|---|---|---|")
+    print("\n".join(rows))
+
+
+def _darotar_kernels(width, heads, ff, tokens, batch, context, timed, pk):
+    """The table rows of :func:`case_darotar`: its kernels and their like kernels alone."""
+    import torch
+
+    from hi_b200.kernels import ops
+
+    bf, f32, hd, nkv, inter = torch.bfloat16, torch.float32, 128, max(1, heads // 4), ff // 2
+    dg = torch.Generator(device=DEV).manual_seed(0)
+    rnd = lambda *shape, dt=bf: torch.randn(*shape, device=DEV, generator=dg).to(dt)
+    rows = []
+
+    def row(kind, name, ms, nbytes, note=""):
+        rows.append(f"| {kind} | {name} | {ms * 1e3:.1f} | {nbytes / 1e6:.1f} | {nbytes / ms / 1e6:,.0f} | "
+                    f"{nbytes / ms / 1e6 / pk['hbm_gbs']:.2f} | {note} |")
+
+    inv = torch.tensor([10000.0 ** (-2.0 * i / hd) for i in range(hd // 2)], device=DEV)
+    inv_r = torch.tensor([500000.0 ** (-2.0 * i / 64) for i in range(32)], device=DEV)
+    for n, seqs, ctx_len, what in ((tokens, 1, tokens, "prefill"), (batch, batch, context, "decode")):
+        single = seqs == n
+        cu = torch.arange(0, n + 1, n // seqs, dtype=torch.int32, device=DEV)
+        sot = torch.repeat_interleave(torch.arange(seqs, device=DEV), n // seqs).to(torch.int32)
+        per = -(-ctx_len // PAGE)
+        pos = (torch.full((n,), ctx_len - 1, device=DEV) if single else torch.arange(n, device=DEV)).to(torch.int32)
+        table = torch.randperm(seqs * per, device=DEV, generator=dg).to(torch.int32).view(seqs, per).contiguous()
+        # boundaries
+        x, d, w1, wb = rnd(n, width, dt=f32), rnd(n, width), rnd(width, dt=f32), rnd(width)
+        routed, slot = rnd(2 * n, width, dt=f32), torch.randperm(2 * n, device=DEV, generator=dg).to(torch.int32)
+        row(what, "boundary: norm of the result, sum, the stream's rounding",
+            timed(lambda: ops.sandwich_step(x, w1, 1e-5, delta=d, out_dtype=bf)), n * width * 12)
+        row(what, "like: residual add + RMSNorm", timed(lambda: ops.add_rmsnorm(x, d, wb, 1e-5, bf)), n * width * 12)
+        row(what, "boundary of two routed rows a token",
+            timed(lambda: ops.sandwich_step(x, w1, 1e-5, routed=routed, slot_of_entry=slot, top_k=2, out_dtype=bf)), n * width * 18)
+        row(what, "like: residual add + RMSNorm of the same",
+            timed(lambda: ops.add_rmsnorm(x, None, wb, 1e-5, bf, None, False, routed, slot, 2)), n * width * 18)
+        # q and k
+        kp, vp = rnd(seqs * per, nkv, PAGE, hd), rnd(seqs * per, nkv, PAGE, hd)
+        qkv, qk = rnd(n, (heads + 2 * nkv) * hd), rnd(n, (heads + nkv) * hd)
+        enc = lambda t, same: ops.qkv_post(t, heads, nkv, hd, pos, inv, True, True, 1e-5, None, sot, table, kp, vp, PAGE, True,
+                                           values_are_keys=same)
+        row(what, "q/k: rotation, norm, append of keys that are values", timed(lambda: enc(qk, True)), n * (2 * heads + 3 * nkv) * hd * 2)
+        row(what, "like: q/k/v with values of their own", timed(lambda: enc(qkv, False)), n * (2 * heads + 4 * nkv) * hd * 2)
+        # windowed attention
+        q = enc(qk, True)
+        pairs = n * ctx_len if single else n * (n + 1) // 2
+        kv = (n if single else 1) * ctx_len * nkv * hd * 4 + n * heads * hd * 4
+        tf = lambda ms, f: f"{pairs * heads * f / ms / 1e9:,.1f} TFLOP/s"
+        if single:
+            row(what, "windowed attention: decode kernel and merge (the kernel of every window)",
+                timed(lambda: ops.decode_attention(q, kp, vp, table, sot, pos, 0, context, hd ** -0.5, ctx_len)), kv)
+            row(what, "like: without a window (TMA tiles)",
+                timed(lambda: ops.decode_attention(q, kp, vp, table, sot, pos, 0, 0, hd ** -0.5, ctx_len)), kv)
+            one = lambda t, same: ops.decode_attention_fused(t, heads, nkv, hd, pos, inv, True, True, 1e-5, None, sot, table, kp, vp, 0, 0,
+                                                             hd ** -0.5, ctx_len, values_are_keys=same)
+            row(what, "no window: encoding, append, attention, merge in one launch, keys that are values", timed(lambda: one(qk, True)), kv)
+            row(what, "like: with values of their own", timed(lambda: one(qkv, False)), kv)
+        else:
+            ms = timed(lambda: ops.prefill_attention_tc(q, kp, vp, table, cu, pos, 1, n, 0, 4096, hd ** -0.5))
+            row(what, "windowed attention: tcgen05 prefill", ms, kv, tf(ms, 4 * hd))
+            ms = timed(lambda: ops.prefill_attention_tc(q, kp, vp, table, cu, pos, 1, n, 0, 0, hd ** -0.5))
+            row(what, "like: without a window", ms, kv, tf(ms, 4 * hd))
+        # latent attention
+        lat, wl = rnd(n, 192), rnd(128)
+        pool, sinks = rnd(seqs * per, 1, PAGE, 192), rnd(heads, dt=f32)
+        row(what, "latent: RMS norm + rotated key part into its page", timed(lambda: ops.latent_append(lat, wl, 1e-5, pos, sot, table, pool, inv_freq=inv_r)), n * 192 * 4)
+        ql = rnd(n, heads, 192)
+        lb = (n if single else 1) * ctx_len * 384 + n * heads * 768
+        for label, kw in (("latent attention over rows of 192 with a learned sink", {"sink_values": sinks}), ("like: without a sink", {})):
+            if single:
+                row(what, label + ": decode kernel and merge", timed(lambda: ops.decode_attention(ql, pool, pool, table, sot, pos, 0, 0, 192 ** -0.5, ctx_len, **kw)), lb)
+            else:
+                ms = timed(lambda: ops.prefill_attention_tc(ql, pool, pool, table, cu, pos, 1, n, 0, 0, 192 ** -0.5, **kw))
+                row(what, label + ": tcgen05 prefill", ms, lb, tf(ms, 4 * 192))
+        o, gate, hg = rnd(n, heads, 128), rnd(n, heads * 128 + width // 2 + 192)[:, width // 2: width // 2 + heads * 128], rnd(n, heads)
+        row(what, "output gate per element", timed(lambda: ops.gate_rows(o, gate, 128)), n * heads * 128 * 6)
+        row(what, "like: output gate per head", timed(lambda: ops.head_gate(o, hg)), n * heads * 128 * 4)
+        # experts
+        rwt, wg, wu = rnd(8, width), rnd(8, inter, width), rnd(8, inter, width)
+        row(what, "router on the stream itself, plan", timed(lambda: ops.router_plan(x, rwt, 2)), n * width * 4)
+        _i, scores, plan = ops.router_plan(x, rwt, 2)
+        xb, ones = x.to(bf), torch.ones(n, 2, device=DEV)
+        for label, sc in (("experts' gate/up of scored inputs, tcgen05", scores), ("like: inputs as they are", ones)):
+            ms = timed(lambda: ops.moe_gate_up_tc(xb, plan, 2, wg, wu, sc, 0.0))
+            row(what, label, ms, 2 * wg.numel() * 2 + 2 * n * (width + inter) * 2, f"{2 * n * 2 * inter * width * 2 / ms / 1e9:,.1f} TFLOP/s")
+    ops.check_tc_status()
+    return rows
+
+
+def case_darotar_step(tokens=2048, batch=8, context=4096, width=2048, heads=16, ff=8192, layers=3):
+    """One Darotar prompt step and two decode steps with every kernel launched on its own (no captured graph), three
+    layers (latent attention, windowed attention, latent attention over the first one's latents): for a launch list
+    under ncu."""
+    import torch
+
+    from hi_b200.engine.core import Engine, StepEntry
+
+    eng = Engine.from_config(_darotar_config(width, heads, ff, layers), seed=0, dtype="bfloat16", device=DEV, kv_page_size=PAGE,
+                             kv_cache_tokens=batch * (context + 256) + tokens + 256, max_active_requests=batch + 1,
+                             use_cuda_graphs=False)
+    g = torch.Generator().manual_seed(0)
+    for rep in range(2):
+        eng.step([StepEntry("p", torch.randint(0, eng.vocab_size, (tokens,), generator=g).tolist(), [tokens - 1])])
+        eng.finish("p")
+    for i in range(batch):
+        eng.assume_cached(i, context)
+    for _ in range(3):
+        eng.step([StepEntry(i, [int(torch.randint(0, eng.vocab_size, (1,), generator=g))], [0]) for i in range(batch)])
+    torch.cuda.synchronize()
+
+
 # --------------------------------------------------------------------------- Fidatar beside the closest existing models
 def _fidatar_config(width, heads, ff, layers, vocab=32000, chunk=8192):
     """Layers in turn attention (heads of 128, a quarter as many key heads, chunks of 8,192, half of a head
@@ -1948,7 +2139,8 @@ CASES = {"sweep": case_sweep, "decode_timeline": case_decode_timeline, "prefill_
          "vinurax_step": case_vinurax_step, "fidatar": case_fidatar, "fidatar_step": case_fidatar_step,
          "mlstm_recurrence": case_mlstm_recurrence, "surinex": case_surinex, "surinex_step": case_surinex_step,
          "bezasun": case_bezasun, "bezasun_step": case_bezasun_step, "bezasun_attention": case_bezasun_attention,
-         "fofisun": case_fofisun, "fofisun_step": case_fofisun_step}
+         "fofisun": case_fofisun, "fofisun_step": case_fofisun_step,
+         "darotar": case_darotar, "darotar_step": case_darotar_step}
 
 
 if __name__ == "__main__":
