@@ -146,6 +146,34 @@ __global__ void gate_rows_kernel(const T* __restrict__ o, long long o_stride, co
   }
 }
 
+__device__ __forceinline__ void put8(float* p, const float (&v)[8]) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void put8(__nv_bfloat16* p, const float (&v)[8]) {
+  alignas(16) __nv_bfloat162 h[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+  *reinterpret_cast<uint4*>(p) = *reinterpret_cast<uint4*>(h);
+}
+
+// The same, eight neighbouring values a thread: head sizes and strides multiples of eight, rows on 16 bytes. Grid
+// (blocks over a row's eights, rows).
+template <typename T>
+__global__ void gate_rows8_kernel(const T* __restrict__ o, long long o_stride, const T* __restrict__ gate, long long gate_stride,
+                                  T* __restrict__ out, int heads, int hd, int vdim) {
+  const size_t r = blockIdx.y;
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+  if (c >= heads * vdim) return;
+  const int h = c / vdim;
+  float x[8], g[8];
+  hb::load8(o + r * o_stride + (size_t)h * hd + (c - h * vdim), x);
+  hb::load8(gate + r * gate_stride + c, g);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) x[i] /= 1.f + expf(-g[i]);
+  put8(out + r * (size_t)heads * vdim + c, x);
+}
+
 }  // namespace
 
 // part_acc [n_rows][2 * heads][splits][hd], part_ml [n_rows][2 * heads][splits][2] -> out [.][heads][vdim]
@@ -187,6 +215,19 @@ extern "C" int hb_gate_rows(const void* o, long long o_stride, const void* gate,
                             long long rows, int heads, int hd, int vdim, cudaStream_t stream) {
   if (!o || !gate || !out || rows < 0 || heads <= 0 || hd <= 0 || vdim <= 0 || vdim > hd) return HB_ERR_BAD_ARG;
   if (rows == 0) return HB_OK;
+  const bool wide = hd % 8 == 0 && vdim % 8 == 0 && o_stride % 8 == 0 && gate_stride % 8 == 0 && rows <= 65535 &&
+                    (reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) % 16 == 0;
+  if (wide && (dtype == HB_DTYPE_F32 || dtype == HB_DTYPE_BF16)) {
+    const int eights = heads * vdim / 8, threads = eights >= 256 ? 256 : (eights + 31) / 32 * 32;
+    const dim3 grid((eights + threads - 1) / threads, (unsigned)rows);
+    if (dtype == HB_DTYPE_F32)
+      gate_rows8_kernel<float><<<grid, threads, 0, stream>>>((const float*)o, o_stride, (const float*)gate, gate_stride, (float*)out, heads, hd, vdim);
+    else
+      gate_rows8_kernel<__nv_bfloat16><<<grid, threads, 0, stream>>>((const __nv_bfloat16*)o, o_stride, (const __nv_bfloat16*)gate, gate_stride,
+                                                                     (__nv_bfloat16*)out, heads, hd, vdim);
+    HB_LAUNCH_CHECK();
+    return HB_OK;
+  }
   const long long want = (rows * heads * vdim + 255) / 256;
   const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
   if (dtype == HB_DTYPE_F32)

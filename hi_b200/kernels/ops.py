@@ -1088,7 +1088,8 @@ def sigmoid_merge(part_acc: torch.Tensor, positions: torch.Tensor, out_dtype: to
 def sigmoid_attention_tc_supported(q_dtype: torch.dtype, nh: int, nkv: int, hd: int, page_size: int) -> bool:
     """Shapes the tensor-core kernels take with sigmoid weights: those of the decode kernel and of the tcgen05
     prefill kernel at once."""
-    return decode_attention_supported(q_dtype, nh, nkv, hd) and prefill_attention_tc_supported(q_dtype, nh, nkv, hd, page_size)
+    return decode_attention_supported(q_dtype, nh, nkv, hd) and nh // nkv <= 16 and \
+        prefill_attention_tc_supported(q_dtype, nh, nkv, hd, page_size)
 
 
 def sigmoid_decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
@@ -1190,10 +1191,10 @@ def _decode_splits(longest: int, groups: int) -> Tuple[int, int]:
 TC_ROW_LENGTHS = (64, 128, 192)
 
 
-def decode_attention_supported(q_dtype: torch.dtype, nh: int, nkv: int, hd: int, row_tiles: bool = False) -> bool:
-    """Shapes the tensor-core decode kernel takes; anything else goes to the general kernel. ``row_tiles``: more
-    than 16 query heads on a kv head are taken in tiles of 16 (by the kernel that loads its tiles by cp.async)."""
-    return q_dtype == torch.bfloat16 and hd in TC_ROW_LENGTHS and nh % nkv == 0 and (row_tiles or nh // nkv <= 16)
+def decode_attention_supported(q_dtype: torch.dtype, nh: int, nkv: int, hd: int) -> bool:
+    """Shapes the tensor-core decode kernels take; anything else goes to the general kernel. More than 16 query heads
+    on a kv head are taken in tiles of 16 (by the kernel that loads its tiles by cp.async)."""
+    return q_dtype == torch.bfloat16 and hd in TC_ROW_LENGTHS and nh % nkv == 0
 
 
 def decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, block_table: torch.Tensor,
@@ -1212,7 +1213,7 @@ def decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
     _, nkv, page_size, hd2 = k_pages.shape
     if hd2 != hd or k_pages.shape != v_pages.shape:
         raise KernelError("cache pages do not match the query's head_dim")
-    if not decode_attention_supported(q.dtype, nh, nkv, hd, row_tiles=parts):
+    if not decode_attention_supported(q.dtype, nh, nkv, hd):
         raise KernelError(f"decode attention does not take nh={nh} nkv={nkv} head_dim={hd}")
     longest = max(int(max_context), 1)
     if chunk > 0:

@@ -45,23 +45,11 @@ def attend_over_pages(q, k_pages, v_pages, block_table, ctx, nh: int, nkv: int, 
     ``slopes`` (float32 [nh]): slopes[head] * (distance to the key) is taken off after the cap.
     ``keep``: first tokens of a request that a sliding window keeps."""
     positions = ctx.positions
-    # the decode kernel packs the query heads of one kv head into a 16-row tile; more heads on ONE shared kv
-    # head go through it sixteen at a time
-    per_call = nh if nkv > 1 or nh <= 16 else 16
-    decode_ok = ops.decode_attention_supported(q.dtype, per_call, nkv, hd)
+    decode_ok = ops.decode_attention_supported(q.dtype, nh, nkv, hd)
 
     def decode(rows_q, seq, pos, longest):
-        if per_call == nh:
-            return ops.decode_attention(rows_q, k_pages, v_pages, block_table, seq, pos, chunk, sliding, scale, longest,
-                                        sink=sink, softcap=softcap, slopes=slopes, sink_values=sink_values, keep=keep)
-        out = torch.empty_like(rows_q)
-        for first in range(0, nh, per_call):
-            part = rows_q[:, first: first + per_call].contiguous()
-            own = [None if t is None else t[first: first + per_call].contiguous() for t in (slopes, sink_values)]
-            out[:, first: first + per_call] = ops.decode_attention(part, k_pages, v_pages, block_table, seq, pos, chunk,
-                                                                   sliding, scale, longest, sink=sink, softcap=softcap,
-                                                                   slopes=own[0], sink_values=own[1], keep=keep)
-        return out
+        return ops.decode_attention(rows_q, k_pages, v_pages, block_table, seq, pos, chunk, sliding, scale, longest,
+                                    sink=sink, softcap=softcap, slopes=slopes, sink_values=sink_values, keep=keep)
 
     if ctx.max_new == 1 and decode_ok:
         # every token of the step is one request's decoded token: the tensor-core kernel
@@ -102,7 +90,7 @@ def differential_attend_over_pages(q, k_pages, v_pages, block_table, ctx, chunk:
     n, nh, hd = q.shape
     nkv, positions = k_pages.shape[1], ctx.positions
     finish = (lam, eps, mul, vdim, gate)
-    decode_ok = ops.decode_attention_supported(q.dtype, nh, nkv, hd, row_tiles=True)
+    decode_ok = ops.decode_attention_supported(q.dtype, nh, nkv, hd)
 
     def decode(rows_q, seq, pos, longest):
         return ops.decode_attention(rows_q, k_pages, v_pages, block_table, seq, pos, chunk, sliding, scale, longest,

@@ -116,6 +116,42 @@ def test_boundary_that_hands_on_the_stream(width, dt, routed):
     assert h.dtype == dt and torch.equal(h, stream.to(dt)) and (dt == torch.bfloat16 or h is stream)
 
 
+@pytest.mark.parametrize("dt,tol", [(torch.float32, 1e-6), (torch.bfloat16, 8e-3)])
+@pytest.mark.parametrize("rows,heads,hd,vdim,before", [(5, 3, 16, 16, 8), (70, 16, 128, 128, 64), (9, 4, 64, 24, 16), (7, 3, 5, 5, 2),
+                                                       (3, 2, 16, 12, 8), (1, 40, 64, 64, 1)])
+def test_gate_of_every_element(dt, tol, rows, heads, hd, vdim, before):
+    """The gate is a column slice behind ``before`` other columns: aligned and not."""
+    o, proj = rnd(rows, heads, hd, seed=1).to(dt), rnd(rows, before + heads * vdim + 8, seed=2, std=2.0).to(dt)
+    gate = proj.to(DEV)[:, before: before + heads * vdim]
+    want = o[:, :, :vdim].double().reshape(rows, -1) * torch.sigmoid(proj[:, before: before + heads * vdim].double())
+    close(ops().gate_rows(o.to(DEV), gate, vdim), want, tol)
+
+
+@pytest.mark.parametrize("nh,nkv,window", [(40, 2, 0), (40, 2, 100), (34, 2, 0)])
+def test_decode_attention_with_more_than_a_row_tile_of_heads(nh, nkv, window):
+    """More than 16 query heads on a key head, values apart from keys, one split and many: against the plain softmax."""
+    o, dt, page, hd, total = ops(), torch.bfloat16, 64, 128, 1500
+    k, v = rnd(2, total, nkv, hd, seed=1).to(dt), rnd(2, total, nkv, hd, seed=2).to(dt)
+    q, starts = rnd(2, nh, hd, seed=3, std=2.0).to(dt), [total - 1, 70]
+    blocks = -(-total // page)
+    bt = torch.randperm(2 * blocks, generator=torch.Generator().manual_seed(4)).to(torch.int32).view(2, blocks)
+    kp, vp = torch.zeros(2 * blocks, nkv, page, hd, dtype=dt), torch.zeros(2 * blocks, nkv, page, hd, dtype=dt)
+    want = []
+    for i, at in enumerate(starts):
+        for b in range(blocks):
+            part = slice(b * page, min(total, (b + 1) * page))
+            kp[int(bt[i, b]), :, : part.stop - part.start] = k[i, part].transpose(0, 1)
+            vp[int(bt[i, b]), :, : part.stop - part.start] = v[i, part].transpose(0, 1)
+        lo, seen = max(0, at + 1 - window) if window else 0, []
+        for a in range(nh):
+            kd, vd = (t[i, lo: at + 1, a // (nh // nkv)].double() for t in (k, v))
+            seen.append(torch.softmax(kd @ q[i, a].double() * 0.1, -1) @ vd)
+        want.append(torch.stack(seen))
+    got = o.decode_attention(q.to(DEV), kp.to(DEV), vp.to(DEV), bt.to(DEV), torch.arange(2, dtype=torch.int32, device=DEV),
+                             torch.tensor(starts, dtype=torch.int32, device=DEV), 0, window, 0.1, total)
+    close(got, torch.stack(want), 1.5e-2)
+
+
 @pytest.mark.parametrize("dt,tol", [(torch.float32, 1e-5), (torch.bfloat16, 2e-2)])
 @pytest.mark.parametrize("hd", [64, 128, 192, 208])
 @pytest.mark.parametrize("heads", [4, 20])

@@ -298,7 +298,7 @@ def test_two_maps_with_norm_and_gate(dt, hd, vdim, heads, nkv, window, keep):
         fin = (lam, eps, mul, vdim, g)
         new = lambda: torch.empty(n, heads * vdim, dtype=dt, device=DEV)
         close(o.diff_merge(*o.paged_attention(*dev, sot.to(DEV), pos.to(DEV), 0, window, scale, 331, keep=keep, parts=True), *fin, new()), want, tol)
-        if not o.decode_attention_supported(dt, 2 * heads, nkv, hd, row_tiles=True):
+        if not o.decode_attention_supported(dt, 2 * heads, nkv, hd):
             continue
         close(o.diff_merge(*o.decode_attention(*dev, sot.to(DEV), pos.to(DEV), 0, window, scale, 331, keep=keep, parts=True), *fin, new()), want, tol)
         close(o.diff_merge(*o.prefill_attention(*dev, cu.to(DEV), pos.to(DEV), 4, 66, 0, window, scale, keep=keep, parts=True), *fin, new()), want, tol)

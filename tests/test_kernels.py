@@ -210,7 +210,7 @@ def test_decode_attention_on_tensor_cores(shape):
     close(got, want, 2e-2, f"decode attention {shape}")
     close(general, want, 2e-2, f"general attention {shape}")
     assert not o.decode_attention_supported(torch.float32, nh, nkv, hd)
-    assert not o.decode_attention_supported(torch.bfloat16, 40, 2, 128) and not o.decode_attention_supported(torch.bfloat16, 4, 2, 48)
+    assert not o.decode_attention_supported(torch.bfloat16, 5, 2, 128) and not o.decode_attention_supported(torch.bfloat16, 4, 2, 48)
 
 
 @pytest.mark.parametrize("shape", [(4, 2, 128, 64, 0, 0), (4, 2, 128, 16, 100, 0), (8, 2, 64, 32, 0, 50),
